@@ -51,16 +51,7 @@ class ConvAttentionConfig:
     def from_dict(cls, d: Dict[str, Any], where: str) -> "ConvAttentionConfig":
         heads, kv_heads, dim, vdim = _heads(d, where)
         rot = d.get("rot") or {}
-        sc = rot.get("scaling")
-        scaling = RopeScaling()
-        if sc:
-            scaling = RopeScaling("yarn", factor=_need(sc, "factor", f"{where}.rot.scaling", float),
-                                  original_max_position_embeddings=_need(sc, "original", f"{where}.rot.scaling", int),
-                                  fast_turns=_need(sc, "fast", f"{where}.rot.scaling", float),
-                                  slow_turns=_need(sc, "slow", f"{where}.rot.scaling", float))
-            if not (scaling.factor > 0 and scaling.original_max_position_embeddings > 0 and scaling.fast_turns > 0
-                    and scaling.slow_turns > 0):
-                raise ConfigError(f"{where}.rot.scaling: factor, original, fast and slow must be positive")
+        scaling = RopeScaling.yarn(rot.get("scaling"), f"{where}.rot.scaling")
         mask = d.get("mask") or {}
         out = cls(heads, kv_heads, dim, vdim, _need(d, "scale", where, float), int(d.get("conv") or 0),
                   int(mask["size"]) if mask.get("size") else None, int(mask.get("keep_first") or 0),

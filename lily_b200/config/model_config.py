@@ -61,6 +61,22 @@ class RopeScaling:
     table_stretch_slope: float = 0.1
 
     @classmethod
+    def yarn(cls, d: Optional[Dict[str, Any]], where: str) -> "RopeScaling":
+        """The scaling from a config's {factor, original, fast, slow}; none of it: no scaling."""
+        if not d:
+            return cls()
+        try:
+            out = cls("yarn", factor=float(d["factor"]), original_max_position_embeddings=int(d["original"]),
+                      fast_turns=float(d["fast"]), slow_turns=float(d["slow"]))
+        except KeyError as e:
+            raise ConfigError(f"config.json lacks {where}.{e.args[0]}") from None
+        except (TypeError, ValueError):
+            raise ConfigError(f"{where}: factor, original, fast and slow are numbers") from None
+        if not (out.factor > 0 and out.original_max_position_embeddings > 0 and out.fast_turns > 0 and out.slow_turns > 0):
+            raise ConfigError(f"{where}: factor, original, fast and slow must be positive")
+        return out
+
+    @classmethod
     def from_dict(cls, d: Optional[Dict[str, Any]]) -> "RopeScaling":
         if not d:
             return cls()

@@ -2,18 +2,23 @@
 // grouped products, and the weighted sum.  Everything stays on the device (no count is read by the host), so a step
 // can be captured in a CUDA graph.
 //
-//   route     z = W_router h (float32); s = softmax(z) over all router outputs; the `top` largest s + correction are
-//             chosen; their weights are s / (sum of the chosen s + 1e-20)
+//   route     z = W_router h (float32); s = softmax(z) over all router outputs, or sigmoid(z) one by one; the `top`
+//             largest s (+ correction) are chosen; their weights are s, or s / (sum of the chosen s + 1e-20).  One more
+//             row of the matrix may follow the outputs': the sigmoid of its product is the token's gate for a shared expert
 //   align     pairs (token, choice) whose expert has weights are grouped by expert: offsets, the pairs in grouped
 //             order, each pair's place there, and the list of (expert, first row) tiles the products run over
-//   gate/up   a[row, n] = g sigmoid(alpha g) (u + 1), g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit)
+//   gate/up   a[row, n] = g sigmoid(alpha g) (u + 1), g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit), or
+//             silu(g) u with g = W_gate x, u = W_up x; a weight that belongs to the expert's input multiplies g and u
+//             ahead of the activation (both are linear in x)
 //   down      y[row, :] = W_down a[row, :]                                  (float32)
 //   combine   out[t] = sum over the token's choices of weight * (y of the pair, or the token's input itself where the
-//             chosen router output is one of the last `identity` ones, which have no weights)
+//             chosen router output is one of the last `identity` ones, which have no weights); without the weight where
+//             it went into the input; plus gate * the shared expert's output where there is one
 //
 // Each output number of the products is summed over k in a fixed order, so a pair's result does not depend on what
 // else is in the batch.  Router, softmax and the weighted sum are float32.
 #include "common.cuh"
+#include "operand.cuh"
 
 namespace lily {
 
@@ -25,10 +30,11 @@ constexpr int ROUTE_TOP_MAX = 64;
 // A token's logits are summed in the same order whatever TB is.
 template <typename T, int TB>
 __global__ void moe_route_kernel(const T* __restrict__ h, int tokens, int width, const float* __restrict__ router,
-                                 const float* __restrict__ correction, int outputs, int top, int* __restrict__ chosen,
-                                 float* __restrict__ weights) {
+                                 const float* __restrict__ correction, int outputs, int top, int sigmoid, int renormalise,
+                                 int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ gate) {
     __shared__ float picked[4][ROUTE_TOP_MAX];
-    extern __shared__ __align__(16) float dyn[];             // [TB][width] the tokens' rows, then [TB][outputs] their scores
+    extern __shared__ __align__(16) float dyn[];             // [TB][width] the tokens' rows, then [TB][rows of the matrix] their scores
+    const int rows = outputs + (gate ? 1 : 0);
     float* xs = dyn;
     float* sc = dyn + (size_t)TB * width;
     pdl_enter_small();
@@ -57,7 +63,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int tokens, int width,
         for (int i = threadIdx.x; i < TB * width; i += blockDim.x) xs[i] = i < nt * width ? to_float(src[i]) : 0.f;
     }
     __syncthreads();
-    for (int e = warp; e < outputs; e += nwarp) {
+    for (int e = warp; e < rows; e += nwarp) {
         const float* w = router + (size_t)e * width;
         float z[TB];
 #pragma unroll
@@ -96,25 +102,35 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int tokens, int width,
 #pragma unroll
         for (int j = 0; j < TB; ++j) {
             const float total = warp_sum(z[j]);
-            if (lane == 0) sc[j * outputs + e] = total;
+            if (lane == 0) sc[j * rows + e] = total;
         }
     }
     __syncthreads();
-    // softmax and choice: a warp a token
+    // scores and choice: a warp a token
     for (int j = warp; j < nt; j += nwarp) {
-        float* s = sc + j * outputs;
+        float* s = sc + j * rows;
         const int t = t0 + j;
-        float mx = -INFINITY;
-        for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, s[e]);
-        mx = warp_max(mx);
-        float sum = 0.f;
-        for (int e = lane; e < outputs; e += 32) {
-            const float p = expf(s[e] - mx);
-            s[e] = p;
-            sum += p;
+        float inv = 1.f;
+        if (sigmoid) {
+            for (int e = lane; e < rows; e += 32) {
+                const float p = 1.f / (1.f + expf(-s[e]));
+                s[e] = p;
+                if (e == outputs) gate[t] = p;
+            }
+        } else {
+            float mx = -INFINITY;
+            for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, s[e]);
+            mx = warp_max(mx);
+            float sum = 0.f;
+            for (int e = lane; e < outputs; e += 32) {
+                const float p = expf(s[e] - mx);
+                s[e] = p;
+                sum += p;
+            }
+            sum = warp_sum(sum);
+            inv = 1.f / sum;
+            if (gate && lane == 0) gate[t] = 1.f / (1.f + expf(-s[outputs]));
         }
-        sum = warp_sum(sum);
-        const float inv = 1.f / sum;
         __syncwarp();
         float total = 0.f;
         for (int k = 0; k < top; ++k) {
@@ -123,7 +139,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int tokens, int width,
             for (int e = lane; e < outputs; e += 32) {
                 const float p = s[e];
                 if (p < 0.f) continue;                                // taken already
-                const float c = p * inv + correction[e];
+                const float c = correction ? p * inv + correction[e] : p * inv;
                 if (c > best) { best = c; at = e; }
             }
             for (int o = 16; o > 0; o >>= 1) {
@@ -142,7 +158,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int tokens, int width,
             }
             __syncwarp();
         }
-        const float norm = 1.f / (total + 1e-20f);
+        const float norm = renormalise ? 1.f / (total + 1e-20f) : 1.f;
         for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] = picked[warp][k] * norm;
         __syncwarp();
     }
@@ -202,12 +218,20 @@ __global__ void moe_align_kernel(const int* __restrict__ chosen, int pairs, int 
 // the output is the activation in T.  MODE 1: A rows are the rows of `a` in grouped order, the output float32.
 constexpr int EBM = 32, EBN = 64, EBK = 16;
 
+// act 0: the clamped gate; 1: silu(g) u
+__device__ __forceinline__ float expert_gate(int act, float g, float u, float limit, float alpha) {
+    if (act == 1) return (g / (1.f + expf(-g))) * u;
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return (g / (1.f + expf(-alpha * g))) * (u + 1.f);
+}
+
 template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, size_t w_expert, int N, int K,
                 const int* __restrict__ offsets, const int* __restrict__ order, int top,
                 const int* __restrict__ tile_expert, const int* __restrict__ tile_row, const int* __restrict__ tile_count,
-                void* __restrict__ out, float limit, float alpha) {
+                void* __restrict__ out, int act, float limit, float alpha, const float* __restrict__ in_weight) {
     __shared__ float As[EBK][EBM + 4];
     __shared__ float Ws[MODE == 0 ? 2 : 1][EBK][EBN + 4];
     __shared__ int arow[EBM];
@@ -266,9 +290,8 @@ moe_gemm_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, size_
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             if (MODE == 0) {
-                const float g = fminf(acc[i][j], limit);
-                const float u = fminf(fmaxf(acc2[i][j], -limit), limit);
-                ((T*)out)[(size_t)(row0 + r) * N + n] = from_float<T>((g / (1.f + expf(-alpha * g))) * (u + 1.f));
+                const float w = in_weight ? in_weight[order[row0 + r]] : 1.f;
+                ((T*)out)[(size_t)(row0 + r) * N + n] = from_float<T>(expert_gate(act, w * acc[i][j], w * acc2[i][j], limit, alpha));
             } else {
                 ((float*)out)[(size_t)(row0 + r) * N + n] = acc[i][j];
             }
@@ -276,84 +299,114 @@ moe_gemm_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, size_
     }
 }
 
-// grid (tokens, ceil(width / 256)), block 256.  y [pairs in grouped order, width] float32; out [tokens, width] float32.
-template <typename T>
-__global__ void moe_combine_kernel(const float* __restrict__ y, const T* __restrict__ h, const int* __restrict__ place,
-                                   const float* __restrict__ weights, int top, int width, float* __restrict__ out) {
-    pdl_wait();
-    const int t = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
-    if (c >= width) return;
-    float acc = 0.f;
-    for (int k = 0; k < top; ++k) {
-        const int at = place[(size_t)t * top + k];
-        const float w = weights[(size_t)t * top + k];
-        const float v = at >= 0 ? y[(size_t)at * width + c] : to_float(h[(size_t)t * width + c]);
-        acc = fmaf(w, v, acc);
-    }
-    out[(size_t)t * width + c] = acc;
+// out[t] = sum over the token's choices of weight * y[place] (the token's input h where the choice has no weights of its
+// own), the weights left out where `weights` is null, plus gate[t] * shared[t] where `gate` is given.  y [pairs in
+// grouped order, width] in T or float32, out [tokens, width] float32.  grid (tokens, ceil(width / (256 VEC))), block 256.
+template <typename Y> __device__ __forceinline__ float4 four_of(const Y* p);
+template <> __device__ __forceinline__ float4 four_of<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 four_of<__nv_bfloat16>(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(lo.x, lo.y, hi.x, hi.y);
 }
 
+template <typename Y, typename T, int VEC>
+__global__ void moe_combine_kernel(const Y* __restrict__ y, const T* __restrict__ h, const int* __restrict__ place,
+                                   const float* __restrict__ weights, int top, int width, const Operand shared,
+                                   const float* __restrict__ gate, float* __restrict__ out) {
+    pdl_wait();
+    const int t = blockIdx.x, c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+    if (c >= width) return;
+    const size_t at_out = (size_t)t * width + c;
+    if (VEC == 4) {
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k = 0; k < top; ++k) {
+            const int at = place[(size_t)t * top + k];
+            const float w = weights ? weights[(size_t)t * top + k] : 1.f;
+            const float4 v = at >= 0 ? four_of<Y>(y + (size_t)at * width + c) : four_of<T>(h + at_out);
+            acc.x = fmaf(w, v.x, acc.x); acc.y = fmaf(w, v.y, acc.y); acc.z = fmaf(w, v.z, acc.z); acc.w = fmaf(w, v.w, acc.w);
+        }
+        if (gate) {
+            const float g = gate[t];
+            const float4 v = shared.four(at_out);
+            acc.x = fmaf(g, v.x, acc.x); acc.y = fmaf(g, v.y, acc.y); acc.z = fmaf(g, v.z, acc.z); acc.w = fmaf(g, v.w, acc.w);
+        }
+        *reinterpret_cast<float4*>(out + at_out) = acc;
+    } else {
+        float acc = 0.f;
+        for (int k = 0; k < top; ++k) {
+            const int at = place[(size_t)t * top + k];
+            const float w = weights ? weights[(size_t)t * top + k] : 1.f;
+            const float v = at >= 0 ? to_float(y[(size_t)at * width + c]) : to_float(h[at_out]);
+            acc = fmaf(w, v, acc);
+        }
+        if (gate) acc = fmaf(gate[t], shared(at_out), acc);
+        out[at_out] = acc;
+    }
+}
 
 // For the library's grouped product (bfloat16, many rows): the pairs' input rows in grouped order, and the activation
-// over its gate/up result.  grid (pairs), block 128; rows beyond offsets[experts] (pairs without weights) are zeroed
-// so that the product reads nothing unwritten.
-template <typename T>
-__global__ void moe_gather_kernel(const T* __restrict__ h, int width, const int* __restrict__ offsets, int experts,
-                                  const int* __restrict__ order, int top, T* __restrict__ out) {
+// over its gate/up result.  Rows of whole 16-byte pieces (width, ff multiples of 8).  grid (pairs); rows beyond
+// offsets[experts] (pairs without weights) are zeroed so that the product reads nothing unwritten.
+__global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ h, int width, const int* __restrict__ offsets, int experts,
+                                  const int* __restrict__ order, int top, __nv_bfloat16* __restrict__ out) {
     pdl_wait();
     const int row = blockIdx.x;
     const bool live = row < offsets[experts];
-    const T* src = h + (size_t)(live ? order[row] / top : 0) * width;
-    T* dst = out + (size_t)row * width;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = live ? src[c] : from_float<T>(0.f);
+    const uint4* src = reinterpret_cast<const uint4*>(h + (size_t)(live ? order[row] / top : 0) * width);
+    uint4* dst = reinterpret_cast<uint4*>(out + (size_t)row * width);
+    for (int c = threadIdx.x; c < width / 8; c += blockDim.x) dst[c] = live ? src[c] : make_uint4(0, 0, 0, 0);
 }
 
-// a[row, n] = g sigmoid(alpha g) (u + 1) from gu[row] = [gate (ff) | up (ff)], clamped as above.
-template <typename T>
-__global__ void moe_activation_kernel(const T* __restrict__ gu, int ff, T* __restrict__ a, float limit, float alpha) {
+// a[row] = gate(gu[row]) with gu[row] = [gate (ff) | up (ff)], both times the pair's weight first where it belongs to the input.
+__global__ void moe_activation_kernel(const __nv_bfloat16* __restrict__ gu, int ff, __nv_bfloat16* __restrict__ a, int act, float limit,
+                                      float alpha, const float* __restrict__ in_weight, const int* __restrict__ offsets,
+                                      int experts, const int* __restrict__ order) {
     pdl_wait();
     const size_t row = blockIdx.x;
-    for (int n = threadIdx.x; n < ff; n += blockDim.x) {
-        const float g = fminf(to_float(gu[row * 2 * ff + n]), limit);
-        const float u = fminf(fmaxf(to_float(gu[row * 2 * ff + ff + n]), -limit), limit);
-        a[row * ff + n] = from_float<T>((g / (1.f + expf(-alpha * g))) * (u + 1.f));
+    if ((int)row >= offsets[experts]) {                // a row of no pair: the next product must not read what was never written
+        for (int c = threadIdx.x; c < ff / 8; c += blockDim.x) reinterpret_cast<uint4*>(a + row * ff)[c] = make_uint4(0, 0, 0, 0);
+        return;
     }
-}
-
-// out[t] = sum_k weight * (y[place] or h[t]) with y in the activation dtype (the library product's result)
-template <typename T>
-__global__ void moe_combine_rows_kernel(const T* __restrict__ y, const T* __restrict__ h, const int* __restrict__ place,
-                                        const float* __restrict__ weights, int top, int width, float* __restrict__ out) {
-    pdl_wait();
-    const int t = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
-    if (c >= width) return;
-    float acc = 0.f;
-    for (int k = 0; k < top; ++k) {
-        const int at = place[(size_t)t * top + k];
-        const float w = weights[(size_t)t * top + k];
-        const float v = to_float(at >= 0 ? y[(size_t)at * width + c] : h[(size_t)t * width + c]);
-        acc = fmaf(w, v, acc);
+    const float w = in_weight ? in_weight[order[row]] : 1.f;
+    const uint4* gs = reinterpret_cast<const uint4*>(gu + row * 2 * ff);
+    const uint4* us = reinterpret_cast<const uint4*>(gu + row * 2 * ff + ff);
+    for (int c = threadIdx.x; c < ff / 8; c += blockDim.x) {
+        uint4 g4 = gs[c];
+        const uint4 u4 = us[c];
+        __nv_bfloat162* g2 = reinterpret_cast<__nv_bfloat162*>(&g4);
+        const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&u4);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
+            g2[k] = __floats2bfloat162_rn(expert_gate(act, w * g.x, w * u.x, limit, alpha), expert_gate(act, w * g.y, w * u.y, limit, alpha));
+        }
+        reinterpret_cast<uint4*>(a + row * ff)[c] = g4;
     }
-    out[(size_t)t * width + c] = acc;
 }
 
 }  // namespace lily
 
 using namespace lily;
 
+// router [outputs (+ 1 with `gate`), width]; correction [outputs] or null; sigmoid 0: softmax over the outputs, 1: each
+// output's sigmoid; renormalise: the chosen scores over their sum.
 LILY_API int lily_moe_route(const void* h, int tokens, int width, const float* router, const float* correction, int outputs,
-                            int top, int* chosen, float* weights, int dtype, cudaStream_t stream) {
+                            int top, int sigmoid, int renormalise, int* chosen, float* weights, float* gate, int dtype,
+                            cudaStream_t stream) {
     if (tokens == 0) return 0;
     LILY_REQUIRE(outputs >= 1 && outputs <= ROUTE_MAX, "moe_route: %d router outputs (up to %d)", outputs, ROUTE_MAX);
     LILY_REQUIRE(top >= 1 && top <= outputs && top <= ROUTE_TOP_MAX, "moe_route: top %d of %d", top, outputs);
+    const int rows = outputs + (gate ? 1 : 0);
     // four tokens a block once there are blocks enough for the device, and while their rows fit the shared memory
-    const int tb = (tokens >= 1024 && (size_t)(4 * width + 4 * outputs) * sizeof(float) <= 40 * 1024) ? 4 : 1;
-    const size_t smem = (size_t)tb * (width + outputs) * sizeof(float);
+    const int tb = (tokens >= 1024 && (size_t)(4 * width + 4 * rows) * sizeof(float) <= 40 * 1024) ? 4 : 1;
+    const size_t smem = (size_t)tb * (width + rows) * sizeof(float);
     LILY_REQUIRE(width > 0 && smem <= 44 * 1024, "moe_route: rows of %d numbers and %d outputs do not fit a block's shared memory", width, outputs);
     dim3 grid((tokens + tb - 1) / tb), block(128);
 #define GO(T, TB)                                                                                                   \
     launch_pdl(moe_route_kernel<T, TB>, grid, block, smem, stream, (const T*)h, tokens, width, router, correction, outputs, \
-               top, chosen, weights)
+               top, sigmoid, renormalise, chosen, weights, gate)
     if (dtype == kBF16) { if (tb == 4) GO(__nv_bfloat16, 4); else GO(__nv_bfloat16, 1); }
     else { if (tb == 4) GO(float, 4); else GO(float, 1); }
 #undef GO
@@ -373,11 +426,12 @@ LILY_API int lily_moe_align(const int* chosen, int pairs, int experts, int* offs
     return 0;
 }
 
-// mode 0: gate/up with the activation (W [experts, 2 N, K], out [pairs, N] in the activation dtype);
-// mode 1: down (W [experts, N, K], out [pairs, N] float32).
+// mode 0: gate/up with the activation (W [experts, 2 N, K], out [pairs, N] in the activation dtype; in_weight: the pairs'
+// weights where they belong to the input, else null); mode 1: down (W [experts, N, K], out [pairs, N] float32).
 LILY_API int lily_moe_gemm(int mode, const void* A, int lda, const void* W, int N, int K, const int* offsets,
                            const int* order, int top, const int* tile_expert, const int* tile_row, const int* tile_count,
-                           int max_tiles, void* out, float limit, float alpha, int dtype, cudaStream_t stream) {
+                           int max_tiles, void* out, int act, float limit, float alpha, const float* in_weight, int dtype,
+                           cudaStream_t stream) {
     if (max_tiles == 0 || N == 0) return 0;
     LILY_REQUIRE(K > 0 && lda >= K && (mode == 0 || mode == 1), "moe_gemm: mode=%d N=%d K=%d lda=%d", mode, N, K, lda);
     LILY_REQUIRE(max_tiles <= 65535, "moe_gemm: %d tiles", max_tiles);
@@ -385,7 +439,7 @@ LILY_API int lily_moe_gemm(int mode, const void* A, int lda, const void* W, int 
     const size_t w_expert = (size_t)(mode == 0 ? 2 : 1) * N * K;
 #define GO(T, MODE)                                                                                                \
     launch_pdl(moe_gemm_kernel<T, MODE>, grid, block, 0, stream, (const T*)A, lda, (const T*)W, w_expert, N, K, offsets, \
-               order, top, tile_expert, tile_row, tile_count, out, limit, alpha)
+               order, top, tile_expert, tile_row, tile_count, out, act, limit, alpha, in_weight)
     if (dtype == kBF16) { if (mode == 0) GO(__nv_bfloat16, 0); else GO(__nv_bfloat16, 1); }
     else { if (mode == 0) GO(float, 0); else GO(float, 1); }
 #undef GO
@@ -393,54 +447,46 @@ LILY_API int lily_moe_gemm(int mode, const void* A, int lda, const void* W, int 
     return 0;
 }
 
-LILY_API int lily_moe_combine(const float* y, const void* h, const int* place, const float* weights, int tokens, int top,
-                              int width, float* out, int dtype, cudaStream_t stream) {
+// y_dtype: float32 (this file's product) or the activation dtype (the library's); weights null: the pairs' outputs as they
+// are; gate null: no shared expert.
+LILY_API int lily_moe_combine(const void* y, int y_dtype, const void* h, const int* place, const float* weights, int tokens, int top,
+                              int width, const void* shared, int shared_dtype, int shared_splits, size_t shared_stride,
+                              const float* gate, float* out, int dtype, cudaStream_t stream) {
     if (tokens == 0) return 0;
-    dim3 grid(tokens, (width + 255) / 256), block(256);
-    if (dtype == kBF16)
-        launch_pdl(moe_combine_kernel<__nv_bfloat16>, grid, block, 0, stream, y, (const __nv_bfloat16*)h, place, weights, top,
-                   width, out);
-    else
-        launch_pdl(moe_combine_kernel<float>, grid, block, 0, stream, y, (const float*)h, place, weights, top, width, out);
+    LILY_REQUIRE(y_dtype == dtype || y_dtype == kF32, "moe_combine: outputs are the activation dtype or float32");
+    LILY_REQUIRE(!gate || (shared && shared_splits >= 1 && (shared_splits == 1 || shared_dtype == kF32)), "moe_combine: the shared expert's output");
+    const Operand sh{shared, shared_dtype == kBF16, shared_splits, shared_stride};
+    const bool vec = width % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)h & 15) == 0 && ((uintptr_t)out & 15) == 0 && sh.vector_ok();
+    const int per = vec ? 4 : 1;
+    dim3 grid(tokens, (width + 256 * per - 1) / (256 * per)), block(256);
+#define GO(Y, T)                                                                                                             \
+    do {                                                                                                                     \
+        if (vec) launch_pdl(moe_combine_kernel<Y, T, 4>, grid, block, 0, stream, (const Y*)y, (const T*)h, place, weights, top, width, sh, gate, out); \
+        else launch_pdl(moe_combine_kernel<Y, T, 1>, grid, block, 0, stream, (const Y*)y, (const T*)h, place, weights, top, width, sh, gate, out);     \
+    } while (0)
+    if (dtype == kBF16) { if (y_dtype == kF32) GO(float, __nv_bfloat16); else GO(__nv_bfloat16, __nv_bfloat16); }
+    else GO(float, float);
+#undef GO
     LILY_CHECK_LAUNCH("moe_combine");
     return 0;
 }
 
 LILY_API int lily_moe_gather(const void* h, int width, const int* offsets, int experts, const int* order, int top, int pairs,
-                             void* out, int dtype, cudaStream_t stream) {
+                             void* out, cudaStream_t stream) {
     if (pairs == 0) return 0;
-    if (dtype == kBF16)
-        launch_pdl(moe_gather_kernel<__nv_bfloat16>, dim3(pairs), dim3(128), 0, stream, (const __nv_bfloat16*)h, width, offsets,
-                   experts, order, top, (__nv_bfloat16*)out);
-    else
-        launch_pdl(moe_gather_kernel<float>, dim3(pairs), dim3(128), 0, stream, (const float*)h, width, offsets, experts, order,
-                   top, (float*)out);
+    LILY_REQUIRE(width % 8 == 0 && ((uintptr_t)h & 15) == 0 && ((uintptr_t)out & 15) == 0, "moe_gather: rows of %d are not whole 16-byte pieces", width);
+    launch_pdl(moe_gather_kernel, dim3(pairs), dim3(width >= 2048 ? 256 : 128), 0, stream, (const __nv_bfloat16*)h, width, offsets,
+               experts, order, top, (__nv_bfloat16*)out);
     LILY_CHECK_LAUNCH("moe_gather");
     return 0;
 }
 
-LILY_API int lily_moe_activation(const void* gu, int ff, int rows, void* a, float limit, float alpha, int dtype,
-                                 cudaStream_t stream) {
+LILY_API int lily_moe_activation(const void* gu, int ff, int rows, void* a, int act, float limit, float alpha, const float* in_weight,
+                                 const int* offsets, int experts, const int* order, cudaStream_t stream) {
     if (rows == 0) return 0;
-    if (dtype == kBF16)
-        launch_pdl(moe_activation_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, stream, (const __nv_bfloat16*)gu, ff,
-                   (__nv_bfloat16*)a, limit, alpha);
-    else
-        launch_pdl(moe_activation_kernel<float>, dim3(rows), dim3(256), 0, stream, (const float*)gu, ff, (float*)a, limit, alpha);
+    LILY_REQUIRE(ff % 8 == 0 && ((uintptr_t)gu & 15) == 0 && ((uintptr_t)a & 15) == 0, "moe_activation: rows of %d are not whole 16-byte pieces", ff);
+    launch_pdl(moe_activation_kernel, dim3(rows), dim3(ff >= 1024 ? 128 : (ff >= 512 ? 64 : 32)), 0, stream, (const __nv_bfloat16*)gu, ff,
+               (__nv_bfloat16*)a, act, limit, alpha, in_weight, offsets, experts, order);
     LILY_CHECK_LAUNCH("moe_activation");
-    return 0;
-}
-
-LILY_API int lily_moe_combine_rows(const void* y, const void* h, const int* place, const float* weights, int tokens, int top,
-                                   int width, float* out, int dtype, cudaStream_t stream) {
-    if (tokens == 0) return 0;
-    dim3 grid(tokens, (width + 255) / 256), block(256);
-    if (dtype == kBF16)
-        launch_pdl(moe_combine_rows_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)y, (const __nv_bfloat16*)h,
-                   place, weights, top, width, out);
-    else
-        launch_pdl(moe_combine_rows_kernel<float>, grid, block, 0, stream, (const float*)y, (const float*)h, place, weights, top,
-                   width, out);
-    LILY_CHECK_LAUNCH("moe_combine_rows");
     return 0;
 }

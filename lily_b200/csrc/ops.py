@@ -52,7 +52,7 @@ _SIGNATURES = {
     "lily_delta_rule": [_vp, _i, _i, _i, _i, _vp, _i, _i, _i, _vp, _vp, _vp, _sz, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _i, _vp],
     "lily_selective_scan": [_vp, _vp, _i, _i, _i, _vp, _vp, _i, _i, _vp, _vp, _vp, _sz, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp],
     "lily_selective_combine": [_vp, _sz, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _vp],
-    "lily_activation": [_vp, _i, _i, _sz, _vp, _i, _sz, _i, _vp],
+    "lily_activation": [_vp, _i, _i, _sz, _vp, _i, _sz, _i, _f, _f, _vp],
     "lily_diff_prepare": [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _vp],
     "lily_diff_combine": [_vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _f, _f, _f, _i, _vp],
     "lily_ssd_scan": [_vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _sz, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp,
@@ -68,17 +68,16 @@ _SIGNATURES = {
     "lily_wkv_scan": [_vp, _vp, _vp, _i, _vp, _vp, _vp, _sz, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp],
     "lily_wkv_combine": [_vp, _sz, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "lily_group_rmsnorm_gate": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _f, _i, _vp],
-    "lily_latent_prepare": [_vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _vp,
+    "lily_latent_prepare": [_vp, _i, _i, _sz, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _vp,
                             _i, _i, _vp],
-    "lily_latent_query": [_vp, _i, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _vp],
-    "lily_head_gate": [_vp, _i, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp],
-    "lily_moe_route": [_vp, _i, _i, _vp, _vp, _i, _i, _vp, _vp, _i, _vp],
+    "lily_latent_query": [_vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _vp],
+    "lily_head_gate": [_vp, _i, _vp, _i, _i, _sz, _i, _i, _i, _i, _i, _vp, _i, _vp],
+    "lily_moe_route": [_vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp],
     "lily_moe_align": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp],
-    "lily_moe_gemm": [_i, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _f, _f, _i, _vp],
-    "lily_moe_combine": [_vp, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _vp],
-    "lily_moe_gather": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp],
-    "lily_moe_activation": [_vp, _i, _i, _vp, _f, _f, _i, _vp],
-    "lily_moe_combine_rows": [_vp, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _vp],
+    "lily_moe_gemm": [_i, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _i, _f, _f, _vp, _i, _vp],
+    "lily_moe_combine": [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _sz, _vp, _vp, _i, _vp],
+    "lily_moe_gather": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp],
+    "lily_moe_activation": [_vp, _i, _i, _vp, _i, _f, _f, _vp, _vp, _i, _vp, _vp],
     "lily_argmax": [_vp, _vp, _vp, _vp, _i, _i, _vp],
     "lily_apply_penalties": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _vp],
     "lily_top_logprobs": [_vp, _vp, _vp, _vp, _vp, _i, _i, _vp],
@@ -431,21 +430,24 @@ def gemm_tc_takes(x: torch.Tensor, weight: torch.Tensor) -> bool:
 
 def gemm_tc(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
             silu_mul_block: bool = False, activation: str = "silu", plain_activation: Optional[str] = None,
-            limit: float = 0.0, alpha: float = 1.0) -> torch.Tensor:
+            limit: float = 0.0, alpha: float = 1.0, factors: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
     """``x [M, K] . weight [N, K]^T`` in bfloat16 on the tcgen05 tensor cores (TMA-fed, accumulator
     in tensor memory).  With ``silu_mul_block`` the rows of ``weight`` alternate between 128 gate
     rows and the 128 up rows of the same outputs and the result is ``act(gate) * up`` [M, N / 2]
-    (``activation``: "silu", "gelu_tanh", or "swish_clamped" with its ``limit`` and ``alpha``).  ``plain_activation`` ("silu", "gelu_tanh", "relu2"): the plain product
-    with that activation on every output, applied to the float32 sums in the epilogue."""
+    (``activation``: "silu", "gelu_tanh", or "swish_clamped" with its ``limit`` and ``alpha``).  ``plain_activation`` ("silu", "gelu_tanh", "relu2",
+    or "xielu" with its ``factors``): the plain product with that activation on every output, applied to the float32 sums
+    in the epilogue."""
     _dev(x, weight, bias)
     m, k = x.shape
     n = weight.shape[0]
     if not gemm_tc_takes(x, weight) or weight.shape[1] != k:
         raise KernelError(f"gemm_tc: x {tuple(x.shape)} {x.dtype} against weight {tuple(weight.shape)} {weight.dtype}")
     out = torch.empty((m, n // 2 if silu_mul_block else n), dtype=torch.bfloat16, device=x.device)
-    _call("lily_gemm_tc", _p(x), _p(weight), _p(out), _p(bias), m, n, k, k, out.shape[1],
-          (6 if activation == "swish_clamped" else 1 + ACTIVATIONS[activation]) if silu_mul_block
-          else (3 + PLAIN_ACTIVATIONS[plain_activation] if plain_activation else 0), float(limit), float(alpha), _stream())
+    if silu_mul_block:
+        epilogue, p0, p1 = 6 if activation == "swish_clamped" else 1 + ACTIVATIONS[activation], limit, alpha
+    else:
+        epilogue, (p0, p1) = {None: 0, "xielu": 7}.get(plain_activation) or (3 + PLAIN_ACTIVATIONS[plain_activation] if plain_activation else 0), factors
+    _call("lily_gemm_tc", _p(x), _p(weight), _p(out), _p(bias), m, n, k, k, out.shape[1], epilogue, float(p0), float(p1), _stream())
     return out
 
 
@@ -1181,16 +1183,27 @@ def gated_group_rmsnorm(y: torch.Tensor, proj: torch.Tensor, gain: torch.Tensor,
 
 # ------------------------------------------------------------------------------ per-head products
 
-def head_linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+def head_linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
+                out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One product per head: ``x`` [tokens, heads, k] (a view whose last axis is contiguous; the heads may be columns
     of a wider row), ``weight`` [heads, n, k]; returns [heads, tokens, n].  float32: this package's FFMA kernel, a
     head a grid plane; bfloat16: the library's batched product with float32 accumulation (``out_dtype=float32``
-    keeps the accumulator's precision)."""
+    keeps the accumulator's precision).  ``out``: a view [tokens, heads, n] in ``x``'s dtype whose last axis is contiguous
+    (the heads may be columns of a wider row); the product is written there and ``out`` is returned."""
     _dev(weight)
     tokens, heads, k = x.shape
     if not x.is_cuda or x.stride(2) != 1 or weight.shape[0] != heads or weight.shape[2] != k or weight.dtype != x.dtype:
         raise KernelError(f"head_linear: x {tuple(x.shape)} {x.dtype} strides {x.stride()} against weight {tuple(weight.shape)} {weight.dtype}")
     n = weight.shape[1]
+    if out is not None:
+        if not out.is_cuda or tuple(out.shape) != (tokens, heads, n) or out.stride(2) != 1 or out.dtype != x.dtype:
+            raise KernelError(f"head_linear: out {tuple(out.shape)} {out.dtype} strides {out.stride()} for [{tokens}, {heads}, {n}] {x.dtype}")
+        if x.dtype == torch.float32:
+            _call("lily_gemm_fp32_heads", _p(x), _p(weight), _p(out), tokens, n, k, x.stride(0), out.stride(0), heads, x.stride(1), n * k,
+                  out.stride(1), _stream())
+        else:
+            torch.bmm(x.transpose(0, 1), weight.transpose(1, 2), out=out.transpose(0, 1))
+        return out
     if x.dtype == torch.float32:
         out = torch.empty((heads, tokens, n), dtype=torch.float32, device=x.device)
         _call("lily_gemm_fp32_heads", _p(x), _p(weight), _p(out), tokens, n, k, x.stride(0), n, heads, x.stride(1), n * k,
@@ -1351,13 +1364,15 @@ def latent_prepare(down: torch.Tensor, q0: int, q_rank: int, kv0: int, rank: int
                    q_gain: torch.Tensor, kv_gain: torch.Tensor, eps: float, cos: Optional[torch.Tensor],
                    sin: Optional[torch.Tensor], positions: torch.Tensor, token_req: torch.Tensor,
                    block_table: torch.Tensor, layer: torch.Tensor, page_size: int, write_kv: bool = True) -> torch.Tensor:
-    """From a token's row of the stacked down-projection ``down`` (the cache's dtype or float32): the RMS-normed query
+    """From a token's row of the stacked down-projection ``down`` (the cache's dtype, float32, or float32 partial sums
+    [splits, tokens, cols]): the RMS-normed query
     latent (columns ``q0`` on, ``q_rank`` of them, gain ``q_gain``), returned as [tokens, q_rank] in the cache's
     dtype; and into the token's cache row [rank + rot] of ``layer`` [pages, page_size * (rank + rot)] the RMS-normed
     key/value latent (columns ``kv0`` on, gain ``kv_gain``) followed by the ``rot`` columns after it, the first
     ``rotary_dim`` of them rotated in halves by the position's angles."""
     _dev(down, q_gain, kv_gain, cos, sin, positions, token_req, block_table, layer)
-    tokens = down.shape[0]
+    tokens, cols = down.shape[-2:]
+    ptr, dt, splits, stride = _operand(down, tokens, cols, "latent_prepare")
     if layer.dim() != 2 or layer.shape[1] != page_size * (rank + rot):
         raise KernelError(f"latent_prepare: cache layer {tuple(layer.shape)} does not hold pages of {page_size} rows of {rank + rot}")
     if q_gain.dtype != torch.float32 or kv_gain.dtype != torch.float32:
@@ -1365,35 +1380,36 @@ def latent_prepare(down: torch.Tensor, q0: int, q_rank: int, kv0: int, rank: int
     if rotary_dim and (cos is None or cos.dtype != torch.float32 or cos.shape[-1] != rotary_dim // 2):
         raise KernelError("rotation tables must be float32 [positions, rotary_dim / 2]")
     cq = torch.empty((tokens, q_rank), dtype=layer.dtype, device=down.device)
-    _call("lily_latent_prepare", _p(down), _dt(down), down.stride(0), q0, q_rank, kv0, rank, rot, rotary_dim, _p(q_gain),
+    _call("lily_latent_prepare", ptr, dt, splits, stride, cols, q0, q_rank, kv0, rank, rot, rotary_dim, _p(q_gain),
           _p(kv_gain), float(eps), _p(cos), _p(sin), _i32(positions, "positions"), _i32(token_req, "token_req"),
           _i32(block_table, "block_table"), block_table.shape[-1], _p(layer), page_size, int(write_kv), _p(cq), tokens,
           _dt(layer), _stream())
     return cq
 
 
-def latent_query(qa: torch.Tensor, q: torch.Tensor, heads: int, d: int, rank: int, rot: int, rotary_dim: int,
+def latent_query(queries: torch.Tensor, q: torch.Tensor, heads: int, d: int, rank: int, rot: int, rotary_dim: int,
                  cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], positions: torch.Tensor) -> torch.Tensor:
-    """The queries the attention over the latent takes, [tokens, heads * (rank + rot)] in ``q``'s dtype: for each head
-    ``qa[head, token]`` (its unrotated part carried into the latent's space, [heads, tokens, rank], ``q``'s dtype or
-    float32) followed by the last ``rot`` columns of the head in ``q`` [tokens, heads * (d + rot)], rotated."""
-    _dev(qa, q, cos, sin, positions)
+    """Completes ``queries`` [tokens, heads * (rank + rot)], the queries the attention over the latent takes: behind the
+    first ``rank`` columns of each head (its unrotated part carried into the latent's space, which ``head_linear`` has put
+    there) go the last ``rot`` columns of the head in ``q`` [tokens, heads * (d + rot)], rotated."""
+    _dev(queries, q, cos, sin, positions)
     tokens = q.shape[0]
-    if tuple(qa.shape) != (heads, tokens, rank) or q.shape[1] != heads * (d + rot):
-        raise KernelError(f"latent_query: qa {tuple(qa.shape)}, q {tuple(q.shape)}")
-    out = torch.empty((tokens, heads * (rank + rot)), dtype=q.dtype, device=q.device)
-    _call("lily_latent_query", _p(qa), _dt(qa), _p(q), tokens, heads, d, rank, rot, rotary_dim, _p(cos), _p(sin),
-          _i32(positions, "positions"), _p(out), _dt(q), _stream())
-    return out
+    if tuple(queries.shape) != (tokens, heads * (rank + rot)) or q.shape[1] != heads * (d + rot) or q.dtype != queries.dtype:
+        raise KernelError(f"latent_query: queries {tuple(queries.shape)} {queries.dtype}, q {tuple(q.shape)} {q.dtype}")
+    _call("lily_latent_query", _p(q), tokens, heads, d, rank, rot, rotary_dim, _p(cos), _p(sin), _i32(positions, "positions"),
+          _p(queries), _dt(q), _stream())
+    return queries
 
 
 def head_gate(ov: torch.Tensor, gate_rows: torch.Tensor, g0: int, out_dtype: torch.dtype) -> torch.Tensor:
-    """``out[t, h * dv + j] = ov[h, t, j] * sigmoid(gate_rows[t, g0 + h])``: ``ov`` [heads, tokens, dv]."""
+    """``out[t, h * dv + j] = ov[h, t, j] * sigmoid(gate_rows[t, g0 + h])``: ``ov`` [heads, tokens, dv]; ``gate_rows``
+    [tokens, cols] or float32 partial sums [splits, tokens, cols]."""
     _dev(ov, gate_rows)
     heads, tokens, dv = ov.shape
+    cols = gate_rows.shape[-1]
+    ptr, dt, splits, stride = _operand(gate_rows, tokens, cols, "head_gate")
     out = torch.empty((tokens, heads * dv), dtype=out_dtype, device=ov.device)
-    _call("lily_head_gate", _p(ov), _dt(ov), _p(gate_rows), _dt(gate_rows), gate_rows.stride(0), g0, tokens, heads, dv,
-          _p(out), _dt(out), _stream())
+    _call("lily_head_gate", _p(ov), _dt(ov), ptr, dt, splits, stride, cols, g0, tokens, heads, dv, _p(out), _dt(out), _stream())
     return out
 
 
@@ -1415,17 +1431,24 @@ class ExpertRouting:
     tile_count: torch.Tensor
     max_tiles: int
     top: int
+    gate: Optional[torch.Tensor] = None      # float32 [tokens]: the shared expert's gate
 
 
-def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, top: int, experts: int) -> ExpertRouting:
-    """Softmax scores over all router outputs (float32 logits ``router . h``), the ``top`` largest scores + correction
-    chosen, their weights the scores themselves over their sum; then the pairs of the first ``experts`` outputs (those
-    with weights; the rest stand for the identity) grouped by expert."""
+def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, experts: int,
+              scores: str = "softmax", renormalise: bool = True, shared_gate: bool = False) -> ExpertRouting:
+    """Scores of all router outputs (float32 logits ``router . h``; their softmax, or with ``scores`` "sigmoid" each one's
+    sigmoid), the ``top`` largest scores (+ correction) chosen, their weights the scores themselves, over their sum with
+    ``renormalise``; then the pairs of the first ``experts`` outputs (those with weights; the rest stand for the identity)
+    grouped by expert.  ``shared_gate``: the matrix has one more row, the sigmoid of whose product is the token's gate for
+    the shared expert."""
     _dev(h, router, correction)
     tokens, width = h.shape
-    outputs = router.shape[0]
-    if router.dtype != torch.float32 or correction.dtype != torch.float32 or router.shape[1] != width or correction.numel() != outputs:
+    outputs = router.shape[0] - (1 if shared_gate else 0)
+    if (router.dtype != torch.float32 or router.shape[1] != width
+            or (correction is not None and (correction.dtype != torch.float32 or correction.numel() != outputs))):
         raise KernelError("moe_route: router [outputs, width] and correction [outputs] are float32")
+    if scores not in ("softmax", "sigmoid"):
+        raise KernelError(f"moe_route: no scores {scores!r} (have softmax, sigmoid)")
     dev = h.device
     pairs = tokens * top
     tile_rows = int(library().lily_moe_tile_rows())
@@ -1434,12 +1457,13 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, t
     chosen, order, place, offsets, tile_expert, tile_row, tile_count = torch.split(
         ints, [pairs, pairs, pairs, experts + 1, max_tiles, max_tiles, 1])
     weights = torch.empty((tokens, top), dtype=torch.float32, device=dev)
-    _call("lily_moe_route", _p(h), tokens, width, _p(router), _p(correction), outputs, top, _p(chosen), _p(weights), _dt(h),
-          _stream())
+    gate = torch.empty((tokens,), dtype=torch.float32, device=dev) if shared_gate else None
+    _call("lily_moe_route", _p(h), tokens, width, _p(router), _p(correction), outputs, top, int(scores == "sigmoid"), int(renormalise),
+          _p(chosen), _p(weights), _p(gate), _dt(h), _stream())
     _call("lily_moe_align", _p(chosen), pairs, experts, _p(offsets), _p(order), _p(place), _p(tile_expert), _p(tile_row),
           _p(tile_count), max_tiles, _stream())
     return ExpertRouting(chosen.view(tokens, top), weights, offsets, order, place, tile_expert, tile_row, tile_count,
-                         max_tiles, top)
+                         max_tiles, top, gate)
 
 
 _OWN_GROUPED = os.environ.get("LILY_B200_GROUPED_GEMM", "") == "own"
@@ -1452,42 +1476,54 @@ def grouped_library_takes(dtype: torch.dtype, width: int, ff: int) -> bool:
             and not _OWN_GROUPED)
 
 
-def moe_experts(h: torch.Tensor, routing: ExpertRouting, w_gate_up: torch.Tensor, w_down: torch.Tensor, limit: float,
-                alpha: float) -> torch.Tensor:
+EXPERT_ACTIVATIONS = {"swish_clamped": 0, "silu": 1}
+
+
+def moe_experts(h: torch.Tensor, routing: ExpertRouting, w_gate_up: torch.Tensor, w_down: torch.Tensor, limit: float = 0.0,
+                alpha: float = 0.0, activation: str = "swish_clamped", weight_on_input: bool = False,
+                shared: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The chosen experts' outputs summed with their weights, float32 [tokens, width].  ``w_gate_up`` [experts, 2 ff,
     width] (an expert's gate rows, then its up rows), ``w_down`` [experts, width, ff].  An expert computes
-    ``W_down (g sigmoid(alpha g) (u + 1))`` with ``g = min(W_gate h, limit)``, ``u = clamp(W_up h, -limit, limit)``; a
-    choice beyond the experts that have weights contributes ``h`` itself."""
-    _dev(h, w_gate_up, w_down)
+    ``W_down (g sigmoid(alpha g) (u + 1))`` with ``g = min(W_gate h, limit)``, ``u = clamp(W_up h, -limit, limit)``, or, with
+    ``activation`` "silu", ``W_down (silu(W_gate h) (W_up h))``; a choice beyond the experts that have weights contributes
+    ``h`` itself.  ``weight_on_input``: a pair's weight multiplies what its expert is given instead of what it gives.
+    ``shared``: the shared expert's output ([tokens, width], or float32 partial sums), added times ``routing.gate``."""
+    if activation not in EXPERT_ACTIVATIONS:
+        raise KernelError(f"moe_experts: no activation {activation!r}; have {sorted(EXPERT_ACTIVATIONS)}")
+    _dev(h, w_gate_up, w_down, shared)
     tokens, width = h.shape
     r = routing
+    if (shared is None) != (r.gate is None):
+        raise KernelError("moe_experts: a shared expert's output comes with its gate")
     pairs = tokens * r.top
     experts = w_down.shape[0] if w_down.dim() == 3 else 0
     ff = w_down.shape[2] if experts else 0
+    act_code, in_weight = EXPERT_ACTIVATIONS[activation], _p(r.weights) if weight_on_input else None
     if experts and grouped_library_takes(h.dtype, width, ff):
         # bfloat16: the library's grouped product over the rows in grouped order (groups end at offsets[1:])
         ends = r.offsets[1:]
         rows = torch.empty((pairs, width), dtype=h.dtype, device=h.device)
-        _call("lily_moe_gather", _p(h), width, _p(r.offsets), experts, _p(r.order), r.top, pairs, _p(rows), _dt(h), _stream())
+        _call("lily_moe_gather", _p(h), width, _p(r.offsets), experts, _p(r.order), r.top, pairs, _p(rows), _stream())
         gate_up = torch._grouped_mm(rows, w_gate_up.transpose(1, 2), offs=ends)
         act = torch.empty((pairs, ff), dtype=h.dtype, device=h.device)
-        _call("lily_moe_activation", _p(gate_up), ff, pairs, _p(act), float(limit), float(alpha), _dt(h), _stream())
+        _call("lily_moe_activation", _p(gate_up), ff, pairs, _p(act), act_code, float(limit), float(alpha), in_weight, _p(r.offsets),
+              experts, _p(r.order), _stream())
         y = torch._grouped_mm(act, w_down.transpose(1, 2), offs=ends)
-        out = torch.empty((tokens, width), dtype=torch.float32, device=h.device)
-        _call("lily_moe_combine_rows", _p(y), _p(h), _p(r.place), _p(r.weights), tokens, r.top, width, _p(out), _dt(h), _stream())
-        return out
-    y = torch.empty((max(pairs, 1), width), dtype=torch.float32, device=h.device)
-    if experts:
-        if w_gate_up.dtype != h.dtype or w_down.dtype != h.dtype or tuple(w_gate_up.shape) != (experts, 2 * ff, width):
-            raise KernelError(f"moe_experts: weights {tuple(w_gate_up.shape)} / {tuple(w_down.shape)} {w_down.dtype} for inputs {tuple(h.shape)} {h.dtype}")
-        act = torch.empty((max(pairs, 1), ff), dtype=h.dtype, device=h.device)
-        _call("lily_moe_gemm", 0, _p(h), h.stride(0), _p(w_gate_up), ff, width, _p(r.offsets), _p(r.order), r.top,
-              _p(r.tile_expert), _p(r.tile_row), _p(r.tile_count), r.max_tiles, _p(act), float(limit), float(alpha), _dt(h),
-              _stream())
-        _call("lily_moe_gemm", 1, _p(act), ff, _p(w_down), width, ff, _p(r.offsets), _p(r.order), r.top, _p(r.tile_expert),
-              _p(r.tile_row), _p(r.tile_count), r.max_tiles, _p(y), 0.0, 0.0, _dt(h), _stream())
+    else:
+        y = torch.empty((max(pairs, 1), width), dtype=torch.float32, device=h.device)
+        if experts:
+            if w_gate_up.dtype != h.dtype or w_down.dtype != h.dtype or tuple(w_gate_up.shape) != (experts, 2 * ff, width):
+                raise KernelError(f"moe_experts: weights {tuple(w_gate_up.shape)} / {tuple(w_down.shape)} {w_down.dtype} for inputs {tuple(h.shape)} {h.dtype}")
+            act = torch.empty((max(pairs, 1), ff), dtype=h.dtype, device=h.device)
+            _call("lily_moe_gemm", 0, _p(h), h.stride(0), _p(w_gate_up), ff, width, _p(r.offsets), _p(r.order), r.top,
+                  _p(r.tile_expert), _p(r.tile_row), _p(r.tile_count), r.max_tiles, _p(act), act_code, float(limit), float(alpha),
+                  in_weight, _dt(h), _stream())
+            _call("lily_moe_gemm", 1, _p(act), ff, _p(w_down), width, ff, _p(r.offsets), _p(r.order), r.top, _p(r.tile_expert),
+                  _p(r.tile_row), _p(r.tile_count), r.max_tiles, _p(y), 0, 0.0, 0.0, None, _dt(h), _stream())
+    sh = (None, _F32, 1, 0) if shared is None else _operand(shared, tokens, width, "moe_experts shared")
     out = torch.empty((tokens, width), dtype=torch.float32, device=h.device)
-    _call("lily_moe_combine", _p(y), _p(h), _p(r.place), _p(r.weights), tokens, r.top, width, _p(out), _dt(h), _stream())
+    _call("lily_moe_combine", _p(y), _dt(y), _p(h), _p(r.place), None if weight_on_input else _p(r.weights), tokens, r.top, width,
+          *sh, _p(r.gate), _p(out), _dt(h), _stream())
     return out
 
 
@@ -1560,7 +1596,7 @@ def top_logprobs(logits: torch.Tensor, k: torch.Tensor):
 
 # ------------------------------------------------------------------------------ norms on both sides of a sublayer, plain feed-forward
 
-PLAIN_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}
+PLAIN_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu2": 2, "xielu": 3}
 # LILY_B200_FUSED_ACTIVATION=0 keeps the plain feed-forward's activation a pass of its own behind the library product
 _FUSED_ACTIVATION = os.environ.get("LILY_B200_FUSED_ACTIVATION", "1") != "0"
 
@@ -1595,28 +1631,47 @@ def add_normed_rmsnorm(resid: torch.Tensor, delta: torch.Tensor, post_gain: torc
     return out
 
 
-def activation(x: torch.Tensor, out_dtype: torch.dtype, activation: str = "relu2") -> torch.Tensor:
-    """``act(x)`` elementwise: "relu2" (the square of max(., 0)), "silu" or "gelu_tanh"; ``x`` [tokens, cols] in either
-    dtype or float32 partial sums [splits, tokens, cols]."""
+def add_normed(resid: torch.Tensor, delta: torch.Tensor, post_gain: torch.Tensor, post_eps: float, mult: float,
+               out_dtype: torch.dtype, normalise: bool = True) -> torch.Tensor:
+    """The add of ``add_normed_rmsnorm`` for a sublayer that reads the stream itself: ``resid`` is updated in place and its
+    new rows come back in ``out_dtype`` (float32: ``resid`` itself), written in the same pass."""
+    _dev(resid, delta, post_gain)
+    n, width = resid.shape
+    if resid.dtype != torch.float32 or post_gain.dtype != torch.float32 or post_gain.numel() != width:
+        raise KernelError("add_normed: the residual stream and the gain behind the sublayer are float32")
+    ptr, dt, splits, stride = _operand(delta, n, width, "add_normed delta")
+    out = None if out_dtype == torch.float32 else torch.empty((n, width), dtype=out_dtype, device=resid.device)
+    _call("lily_add_normed_rmsnorm", _p(resid), ptr, dt, splits, stride, _p(post_gain), float(post_eps), float(mult), None, _F32, _p(out),
+          _dt(out) if out is not None else _F32, None, n, width, 0.0, 1, int(bool(normalise)), _stream())
+    return resid if out is None else out
+
+
+def activation(x: torch.Tensor, out_dtype: torch.dtype, activation: str = "relu2",
+               factors: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
+    """``act(x)`` elementwise: "relu2" (the square of max(., 0)), "silu", "gelu_tanh", or "xielu" with its two ``factors``
+    (a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below); ``x`` [tokens, cols] in either dtype or float32 partial sums
+    [splits, tokens, cols]."""
     if activation not in PLAIN_ACTIVATIONS:
         raise KernelError(f"no activation {activation!r}; have {sorted(PLAIN_ACTIVATIONS)}")
     _dev(x)
     n, cols = x.shape[-2:]
     ptr, dt, splits, stride = _operand(x, n, cols, "activation")
     out = torch.empty((n, cols), dtype=out_dtype, device=x.device)
-    _call("lily_activation", ptr, dt, splits, stride, _p(out), _dt(out), out.numel(), PLAIN_ACTIVATIONS[activation], _stream())
+    _call("lily_activation", ptr, dt, splits, stride, _p(out), _dt(out), out.numel(), PLAIN_ACTIVATIONS[activation], float(factors[0]),
+          float(factors[1]), _stream())
     return out
 
 
-def linear_activation(x: torch.Tensor, weight: torch.Tensor, activation_name: str = "relu2") -> torch.Tensor:
+def linear_activation(x: torch.Tensor, weight: torch.Tensor, activation_name: str = "relu2",
+                      factors: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
     """``act(x @ weight.T)`` in ``x``'s dtype: for 65 tokens and more in bfloat16 the tcgen05 product with the activation
     in its epilogue (where ``gate_up_fused_pays``: the [tokens, N] intermediate is never written); else the product
     (whole, or float32 partial sums for a few tokens) with the activation as a pass over it."""
     if activation_name not in PLAIN_ACTIVATIONS:
         raise KernelError(f"no activation {activation_name!r}; have {sorted(PLAIN_ACTIVATIONS)}")
     if _FUSED_ACTIVATION and gate_up_fused_pays(x.shape[0], weight.shape[0]) and gemm_tc_takes(x, weight) and weight.is_contiguous():
-        return gemm_tc(x, weight, plain_activation=activation_name)
-    return activation(linear_auto(x, weight), x.dtype, activation_name)
+        return gemm_tc(x, weight, plain_activation=activation_name, factors=factors)
+    return activation(linear_auto(x, weight), x.dtype, activation_name, factors)
 
 
 # ------------------------------------------------------------------------------ differential attention

@@ -4,8 +4,10 @@
 //                                                                                         `normalise` 0, u = delta * gain_post: a gain
 //                                                                                         per column alone, a layer scale)
 //                        v = resid + mult * u;  resid = v (when asked)                   (the add, float32)
-//                        out = v / sqrt(mean(v^2) + eps) * weight                        (the norm ahead of the next one)
-//   activation:          out = act(in), act = SiLU, the tanh form of GELU, or the square of max(., 0)
+//                        out = v / sqrt(mean(v^2) + eps) * weight                        (the norm ahead of the next one; or,
+//                                                                                         without `weight`, out = v: a sublayer
+//                                                                                         that reads the stream itself)
+//   activation:          out = act(in), act = SiLU, the tanh form of GELU, the square of max(., 0), or xIELU
 //
 // `delta` and `in` may be the activation dtype, float32, or the float32 partial sums of a split-k product.  Sums of
 // squares, roots and the residual stream are float32 whatever the activation dtype.
@@ -22,9 +24,9 @@ struct NormedAddArgs {
     float* resid;             // [tokens, hidden]
     Operand delta;            // [tokens, hidden]
     const float* post_gain;   // [hidden]
-    const void* weight;       // [hidden], float32 or bfloat16; null: no output, the add alone
+    const void* weight;       // [hidden], float32 or bfloat16; null: the output, where there is one, is the new stream itself
     int weight_bf16;
-    void* out;                // [rows or tokens, hidden]
+    void* out;                // [rows or tokens, hidden]; null: the add alone
     const int* rows;          // null: every token; else the tokens whose output is wanted (nothing is written back then)
     int hidden;
     float post_eps, eps, mult;
@@ -83,9 +85,15 @@ __global__ void add_normed_rmsnorm_kernel(const NormedAddArgs a) {
             ssq = fmaf(v, v, ssq);
         }
     }
-    if (a.weight == nullptr) return;
-    const float inv = rsqrtf(block_sum(ssq, red) / (float)hidden + a.eps);
+    if (a.out == nullptr) return;
     T* dst = (T*)a.out + (size_t)m * hidden;
+    if (a.weight == nullptr) {
+        for (int i = threadIdx.x * VEC; i < hidden; i += blockDim.x * VEC)      // the entries this thread has formed
+#pragma unroll
+            for (int u = 0; u < VEC; ++u) dst[i + u] = from_float<T>(row[i + u]);
+        return;
+    }
+    const float inv = rsqrtf(block_sum(ssq, red) / (float)hidden + a.eps);
     for (int i = threadIdx.x; i < hidden; i += blockDim.x)
         dst[i] = from_float<T>((row[i] * inv) * gain_at(a.weight, a.weight_bf16, i));
 }
@@ -141,9 +149,14 @@ __global__ void add_normed_rmsnorm_reg_kernel(const NormedAddArgs a) {
         if (a.write_residual) *reinterpret_cast<float4*>(a.resid + src + i) = v[k];
         ssq += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
     }
-    if (a.weight == nullptr) return;
-    const float inv = rsqrtf(block_sum_once(ssq, slots[1]) / (float)hidden + a.eps);
+    if (a.out == nullptr) return;
     T* dst = (T*)a.out + (size_t)m * hidden;
+    if (a.weight == nullptr) {
+#pragma unroll
+        for (int k = 0; k < PER; ++k) store_four<T>(dst + (k * blockDim.x + threadIdx.x) * 4, v[k]);
+        return;
+    }
+    const float inv = rsqrtf(block_sum_once(ssq, slots[1]) / (float)hidden + a.eps);
 #pragma unroll
     for (int k = 0; k < PER; ++k) {
         const int i = (k * blockDim.x + threadIdx.x) * 4;
@@ -181,47 +194,56 @@ __global__ void add_normed_rmsnorm_cluster_kernel(const NormedAddArgs a) {
     v.z += a.mult * ((d.z * inv_d) * g.z);
     v.w += a.mult * ((d.w * inv_d) * g.w);
     if (a.write_residual) *reinterpret_cast<float4*>(a.resid + src + i) = v;
+    T* dst = (T*)a.out + (size_t)m * hidden + i;
+    if (a.weight == nullptr) {      // the same in every block of the launch; nothing was sent since the sync above
+        if (a.out != nullptr) {
+            dst[0] = from_float<T>(v.x);
+            dst[1] = from_float<T>(v.y);
+            dst[2] = from_float<T>(v.z);
+            dst[3] = from_float<T>(v.w);
+        }
+        return;
+    }
     mine = block_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w, red);
     if (threadIdx.x < CL) cluster.map_shared_rank(&share[1][0], threadIdx.x)[blockIdx.x] = mine;
     cluster.sync();                 // after it nobody touches another block's shared memory again
-    if (a.weight == nullptr) return;
     total = 0.f;
 #pragma unroll
     for (int r = 0; r < CL; ++r) total += share[1][r];
     const float inv = rsqrtf(total / (float)hidden + a.eps);
-    T* dst = (T*)a.out + (size_t)m * hidden + i;
     dst[0] = from_float<T>((v.x * inv) * gain_at(a.weight, a.weight_bf16, i));
     dst[1] = from_float<T>((v.y * inv) * gain_at(a.weight, a.weight_bf16, i + 1));
     dst[2] = from_float<T>((v.z * inv) * gain_at(a.weight, a.weight_bf16, i + 2));
     dst[3] = from_float<T>((v.w * inv) * gain_at(a.weight, a.weight_bf16, i + 3));
 }
 
-// act: 0 SiLU, 1 the tanh form of GELU, 2 the square of max(., 0)
-__device__ __forceinline__ float activate(int act, float z) {
+// act: 0 SiLU, 1 the tanh form of GELU, 2 the square of max(., 0), 3 xIELU with its two factors
+__device__ __forceinline__ float activate(int act, float z, float p0, float p1) {
+    if (act == 3) return xielu(z, p0, p1);
     if (act == 2) { const float r = fmaxf(z, 0.f); return r * r; }
     if (act == 0) return z / (1.f + expf(-z));
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
 template <typename T, int VEC>
-__global__ void activation_kernel(const Operand in, T* __restrict__ out, size_t total, int act) {
+__global__ void activation_kernel(const Operand in, T* __restrict__ out, size_t total, int act, float p0, float p1) {
     pdl_enter_small();
     const size_t step = (size_t)gridDim.x * blockDim.x * VEC;
     for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC; i < total; i += step) {
         if (VEC == 4) {
             const float4 z = in.four(i);
-            out[i] = from_float<T>(activate(act, z.x));
-            out[i + 1] = from_float<T>(activate(act, z.y));
-            out[i + 2] = from_float<T>(activate(act, z.z));
-            out[i + 3] = from_float<T>(activate(act, z.w));
+            out[i] = from_float<T>(activate(act, z.x, p0, p1));
+            out[i + 1] = from_float<T>(activate(act, z.y, p0, p1));
+            out[i + 2] = from_float<T>(activate(act, z.z, p0, p1));
+            out[i + 3] = from_float<T>(activate(act, z.w, p0, p1));
         } else {
-            out[i] = from_float<T>(activate(act, in(i)));
+            out[i] = from_float<T>(activate(act, in(i), p0, p1));
         }
     }
 }
 
 // bfloat16 in one piece to bfloat16, eight entries a thread and turn (16-byte accesses)
-__global__ void activation_bf16x8_kernel(const __nv_bfloat16* __restrict__ in, __nv_bfloat16* __restrict__ out, size_t total, int act) {
+__global__ void activation_bf16x8_kernel(const __nv_bfloat16* __restrict__ in, __nv_bfloat16* __restrict__ out, size_t total, int act, float p0, float p1) {
     pdl_enter_small();
     const size_t step = (size_t)gridDim.x * blockDim.x * 8;
     for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 8; i < total; i += step) {
@@ -230,7 +252,8 @@ __global__ void activation_bf16x8_kernel(const __nv_bfloat16* __restrict__ in, _
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
             const float2 z = __bfloat1622float2(v2[k]);
-            v2[k] = __floats2bfloat162_rn(activate(act, z.x), activate(act, z.y));
+            v2[k] = act == 3 ? __floats2bfloat162_rn(xielu_fast(z.x, p0, p1), xielu_fast(z.y, p0, p1))
+                             : __floats2bfloat162_rn(activate(act, z.x, p0, p1), activate(act, z.y, p0, p1));
         }
         *reinterpret_cast<uint4*>(out + i) = v;
     }
@@ -314,20 +337,20 @@ LILY_API int lily_add_normed_rmsnorm(float* resid, const void* delta, int delta_
 }
 
 LILY_API int lily_activation(const void* in, int in_dtype, int in_splits, size_t in_stride, void* out, int out_dtype,
-                             size_t total, int act, cudaStream_t stream) {
+                             size_t total, int act, float p0, float p1, cudaStream_t stream) {
     if (total == 0) return 0;
-    LILY_REQUIRE(act >= 0 && act <= 2, "activation: code %d (0 SiLU, 1 GELU tanh, 2 squared ReLU)", act);
+    LILY_REQUIRE(act >= 0 && act <= 3, "activation: code %d (0 SiLU, 1 GELU tanh, 2 squared ReLU, 3 xIELU)", act);
     LILY_REQUIRE(in_splits >= 1 && (in_splits == 1 || in_dtype == kF32), "activation: only float32 partial sums come in several splits");
     const Operand x{in, in_dtype == kBF16, in_splits, in_stride};
     auto blocks_for = [](size_t work) { return (int)((work + 255) / 256 < (size_t)sm_count() * 16 ? (work + 255) / 256 : (size_t)sm_count() * 16); };
     if (in_dtype == kBF16 && out_dtype == kBF16 && total % 8 == 0 && ((uintptr_t)in & 15) == 0 && ((uintptr_t)out & 15) == 0) {
-        launch_pdl(activation_bf16x8_kernel, dim3(blocks_for(total / 8)), dim3(256), 0, stream, (const __nv_bfloat16*)in, (__nv_bfloat16*)out, total, act);
+        launch_pdl(activation_bf16x8_kernel, dim3(blocks_for(total / 8)), dim3(256), 0, stream, (const __nv_bfloat16*)in, (__nv_bfloat16*)out, total, act, p0, p1);
     } else if (total % 4 == 0 && x.vector_ok()) {
-        if (out_dtype == kBF16) launch_pdl(activation_kernel<__nv_bfloat16, 4>, dim3(blocks_for(total / 4)), dim3(256), 0, stream, x, (__nv_bfloat16*)out, total, act);
-        else launch_pdl(activation_kernel<float, 4>, dim3(blocks_for(total / 4)), dim3(256), 0, stream, x, (float*)out, total, act);
+        if (out_dtype == kBF16) launch_pdl(activation_kernel<__nv_bfloat16, 4>, dim3(blocks_for(total / 4)), dim3(256), 0, stream, x, (__nv_bfloat16*)out, total, act, p0, p1);
+        else launch_pdl(activation_kernel<float, 4>, dim3(blocks_for(total / 4)), dim3(256), 0, stream, x, (float*)out, total, act, p0, p1);
     } else {
-        if (out_dtype == kBF16) launch_pdl(activation_kernel<__nv_bfloat16, 1>, dim3(blocks_for(total)), dim3(256), 0, stream, x, (__nv_bfloat16*)out, total, act);
-        else launch_pdl(activation_kernel<float, 1>, dim3(blocks_for(total)), dim3(256), 0, stream, x, (float*)out, total, act);
+        if (out_dtype == kBF16) launch_pdl(activation_kernel<__nv_bfloat16, 1>, dim3(blocks_for(total)), dim3(256), 0, stream, x, (__nv_bfloat16*)out, total, act, p0, p1);
+        else launch_pdl(activation_kernel<float, 1>, dim3(blocks_for(total)), dim3(256), 0, stream, x, (float*)out, total, act, p0, p1);
     }
     LILY_CHECK_LAUNCH("activation");
     return 0;

@@ -19,7 +19,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from lily_b200.parts.attention import LayerCache
-from lily_b200.parts.base import BuildContext, CacheNeed, ModelSpec, RunSlots, StateNeed, TensorSpec, build_part
+from lily_b200.parts.base import BuildContext, CacheNeed, FeedForward, ModelSpec, RunSlots, StateNeed, TensorSpec, build_part
 
 
 class AssembledModel:
@@ -134,6 +134,8 @@ class AssembledModel:
                 if isinstance(v, torch.Tensor) and v.data_ptr() not in seen and not getattr(v, "_is_table", False):
                     seen.add(v.data_ptr())
                     total += v.numel() * v.element_size()
+            for inner in getattr(obj, "parts", ()) if isinstance(obj, FeedForward) else ():
+                visit(inner)                              # a feed-forward put together from others
         visit(self)
         for b in self.blocks:
             for part in b.parts:

@@ -1,6 +1,7 @@
 """Block arrangements.  The pre-norm block: ``r += mixer(norm_in(r)); r += feed_forward(norm_post(r))``; the parallel
 block (``ParallelBlockSpec``): one norm, several mixers and the feed-forward side by side on its output; the sandwich
-block (``SandwichBlockSpec``): a norm on both sides of each sublayer and a multiplier on what enters the stream.
+block (``SandwichBlockSpec``): a norm on both sides of each sublayer and a multiplier on what enters the stream; the
+post-norm block (``PostNormBlockSpec``): a norm behind each sublayer and none ahead of it.
 
 The residual stream ``r`` is float32 and updated in place; each add is fused into the norm that
 follows it, so a block receives the pending delta of the block before it and returns its own
@@ -13,7 +14,7 @@ from dataclasses import dataclass
 from typing import Any, Dict, Tuple
 
 from lily_b200.parts.base import Block, BlockSpec, BuildContext, RunSlots, TensorSpec, build_part, register_part
-from lily_b200.parts.norm import NormedDelta
+from lily_b200.parts.norm import NormedDelta, enter_stream
 
 
 @register_part("block", "prenorm")
@@ -176,3 +177,58 @@ class SandwichBlock(Block):
             return a
         h = self.norm_ff.forward(residual, a)
         return NormedDelta(self.feed_forward.forward(h, batch), self.post_gains[1], eps, mult, divides)
+
+
+@dataclass(frozen=True)
+class PostNormBlockSpec:
+    """A norm behind each sublayer and none ahead of it: ``r += mult * norm_1(mixer(r))``, then, where the block has a
+    feed-forward, ``r += mult * norm_2(ff(r))``.  The sublayers read the stream itself, rounded to the compute dtype; the norm
+    behind a sublayer, the add and that rounding are one pass (``NormedDelta`` with ``enter_stream``), ahead of the next
+    sublayer or, with the final norm, at the end."""
+
+    prefix: str
+    mixer: Any
+    feed_forward: Any                         # None: the block ends behind its mixer
+    norm: Any                                 # the spec of both norms (size, eps, gain naming)
+    mult: float = 1.0
+    kind: str = "postnorm"
+    mixer_name: str = "mix"
+    feed_forward_name: str = "mlp"
+    norm_names: Tuple[str, str] = ("norm1", "norm2")
+
+
+@register_part("block", "postnorm")
+class PostNormBlock(Block):
+    def __init__(self, spec: PostNormBlockSpec, prefix: str, ctx: BuildContext):
+        self.spec, self.ctx = spec, ctx
+        p = spec.prefix
+        self.norm_mixer = build_part("norm", spec.norm, f"{p}.{spec.norm_names[0]}", ctx)
+        self.mixer = build_part("mixer", spec.mixer, f"{p}.{spec.mixer_name}", ctx)
+        self.mixers = (self.mixer,)
+        self.parts = (self.norm_mixer, self.mixer)
+        self.feed_forward = self.norm_ff = None
+        if spec.feed_forward is not None:
+            self.norm_ff = build_part("norm", spec.norm, f"{p}.{spec.norm_names[1]}", ctx)
+            self.feed_forward = build_part("feed_forward", spec.feed_forward, f"{p}.{spec.feed_forward_name}", ctx)
+            self.parts += (self.norm_ff, self.feed_forward)
+        self.gains = []
+
+    def tensors(self) -> Dict[str, TensorSpec]:
+        out: Dict[str, TensorSpec] = {}
+        for part in self.parts:
+            out.update(part.tensors())
+        return out
+
+    def load(self, get) -> None:
+        for part in self.parts:
+            part.load(get)
+        self.gains = [n.weight.float().contiguous() for n in (self.norm_mixer, self.norm_ff) if n is not None]
+
+    def forward(self, residual, delta, batch, run: RunSlots):
+        ops, eps, mult = self.ctx.ops, self.spec.norm.eps, float(self.spec.mult)
+        x = enter_stream(ops, residual, delta, self.ctx.dtype, run.stream_bias)
+        a = NormedDelta(self.mixer.forward(x, batch, run.caches[0], run.states[0], run.write_cache), self.gains[0], eps, mult)
+        if self.feed_forward is None:
+            return a
+        x = enter_stream(ops, residual, a, self.ctx.dtype)
+        return NormedDelta(self.feed_forward.forward(x, batch), self.gains[1], eps, mult)

@@ -5,7 +5,7 @@ Queries go through a latent of their own: ``c_q = rms(W_dq h) * g_q``, ``q = W_u
 RMS-normed with a gain, are the latent ``c``; the rest, rotated by position, are one key part shared by all heads.
 Per head the unrotated key is ``W_uk c`` and the value ``W_uv c``; the score is
 ``(q_unrotated . k_unrotated + q_rotated . k_rotated) * scale`` over the visible positions (all, or the last
-``window``); each head's output is multiplied by ``sigmoid(W_g h)`` of that head, and ``W_o`` closes the part.
+``window``); each head's output is multiplied by ``sigmoid(W_g h)`` of that head (``out_gate``), and ``W_o`` closes the part.
 
 Only ``[c | rotated key part]`` is cached: one row of ``kv_rank + rot_dim`` numbers per position for all heads
 (``CacheNeed`` with one kv head and ``values_in_keys``).  Since ``q_u . (W_uk c) = (W_uk^T q_u) . c``, the unrotated
@@ -14,8 +14,14 @@ then runs over the cached rows as they are, all heads sharing them, with the fir
 values, and ``W_uv`` is applied to each head's weighted sum of latents afterwards (``W_uv sum_j p_j c_j``).  A prompt's
 portion and a decoded token take the same path, so what a position's logits are does not depend on how it arrived.
 
+With ``own_kv`` False the mixer has no ``W_dkv``: it attends to rows that another run's mixer has cached (a schedule entry
+that ``reads`` that run), with its own queries, ``W_uk`` and ``W_uv``.  The two then agree in ``kv_rank``, ``rot_dim`` and
+position encoding.  An interleaved position encoding is served by reordering the rotated rows of ``W_uq`` and ``W_dkv`` once,
+at load time (a score does not change when the columns of query and key are reordered alike).
+
 The three projections that read the mixer's input (query latent, key/value latent, gate) are one product with a
-float32 result; the two RMS norms, the rotation angles, the scores and the softmax are float32 in both precisions.
+float32 result (partial sums for a few tokens); the two RMS norms, the rotation angles, the scores and the softmax are
+float32 in both precisions.  The two products per head write into the rows the next kernel reads, rounded once.
 """
 
 from __future__ import annotations
@@ -27,6 +33,7 @@ import torch
 
 from lily_b200.parts.attention import AttentionPlan, LayerCache
 from lily_b200.parts.base import BuildContext, CacheNeed, Mixer, TensorSpec, build_part, register_part
+from lily_b200.parts.rope import pairing_order
 
 
 @dataclass(frozen=True)
@@ -43,6 +50,7 @@ class LatentAttentionSpec:
     window: Optional[int] = None  # None: all keys; n: the last n keys
     position: Any = None          # a position spec over the rot_dim columns (e.g. RopeSpec) or None
     out_gate: bool = True         # each head's output times sigmoid(W_g h) of the head
+    own_kv: bool = True           # False: the cached rows are another run's; this mixer projects none
     kind: str = "latent_attention"
     # names of the tensors under the part's prefix
     names: Optional[Tuple[Tuple[str, str], ...]] = None
@@ -84,24 +92,43 @@ class LatentAttention(Mixer):
         out = {f"{p}.{s.name('dq')}": TensorSpec((s.q_rank, s.hidden_size)),
                f"{p}.{s.name('dq_norm')}": TensorSpec((s.q_rank,), role="vector", init="gain"),
                f"{p}.{s.name('uq')}": TensorSpec((h * (s.head_dim + s.rot_dim), s.q_rank)),
-               f"{p}.{s.name('dkv')}": TensorSpec((s.row, s.hidden_size)),
-               f"{p}.{s.name('dkv_norm')}": TensorSpec((s.kv_rank,), role="vector", init="gain"),
                f"{p}.{s.name('uk')}": TensorSpec((h * s.head_dim, s.kv_rank)),
                f"{p}.{s.name('uv')}": TensorSpec((h * s.v_head_dim, s.kv_rank)),
                f"{p}.{s.name('o')}": TensorSpec((s.hidden_size, h * s.v_head_dim))}
+        if s.own_kv:
+            out[f"{p}.{s.name('dkv')}"] = TensorSpec((s.row, s.hidden_size))
+            out[f"{p}.{s.name('dkv_norm')}"] = TensorSpec((s.kv_rank,), role="vector", init="gain")
         if s.out_gate:
             out[f"{p}.{s.name('g')}"] = TensorSpec((h, s.hidden_size))
         return out
 
+    def _rotation_order(self) -> Optional[torch.Tensor]:
+        """For an interleaved encoding: the stored row of the rotated part that goes to each place of it."""
+        if self.position is None or not self.position.interleaved:
+            return None
+        return pairing_order(self.spec.rot_dim, self.position.rotary_dim)
+
     def load(self, get) -> None:
         s, p = self.spec, self.prefix
         g = lambda role: get(f"{p}.{s.name(role)}")
-        parts = [g("dq"), g("dkv")] + ([g("g")] if s.out_gate else [])
-        self.w_down = torch.cat(parts, 0).contiguous()                 # [q_rank | kv_rank + rot | heads] rows
+        h, order = s.num_heads, self._rotation_order()
+        parts = [g("dq")]
+        if s.own_kv:
+            dkv = g("dkv")
+            if order is not None:
+                dkv = torch.cat([dkv[:s.kv_rank], dkv[s.kv_rank:][order.to(dkv.device)]], 0)
+            parts.append(dkv)
+        if s.out_gate:
+            parts.append(g("g"))
+        self.w_down = torch.cat(parts, 0).contiguous()                 # [q_rank (| kv_rank + rot) (| heads)] rows
         self.q_gain = g("dq_norm").float().contiguous()
-        self.kv_gain = g("dkv_norm").float().contiguous()
-        self.w_uq = g("uq").contiguous()
-        h = s.num_heads
+        # a mixer that caches nothing has no gain of its own there and reads none
+        self.kv_gain = g("dkv_norm").float().contiguous() if s.own_kv else torch.ones(s.kv_rank, dtype=torch.float32, device=self.q_gain.device)
+        uq = g("uq")
+        if order is not None:
+            uq = uq.view(h, s.head_dim + s.rot_dim, s.q_rank)
+            uq = torch.cat([uq[:, :s.head_dim], uq[:, s.head_dim:][:, order.to(uq.device)]], 1).reshape(-1, s.q_rank)
+        self.w_uq = uq.contiguous()
         # per head [out, in]: q' = W_uk^T q_u takes W_uk^T [kv_rank, head_dim]; the value takes W_uv [v, kv_rank] as stored
         self.w_uk = g("uk").view(h, s.head_dim, s.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = g("uv").view(h, s.v_head_dim, s.kv_rank).contiguous()
@@ -134,15 +161,18 @@ class LatentAttention(Mixer):
         plan = self._plan(batch, cache.group, cache.data.dtype, page)
         cos, sin = self.position.tables() if self.position is not None else (None, None)
         rotary_dim = self.position.rotary_dim if self.position is not None else 0
-        down = ops.linear(x, self.w_down, out_dtype=torch.float32)      # [tokens, q latent | kv latent | rotated | gates]
+        down = ops.linear_split(x, self.w_down)                 # [tokens, q latent (| kv latent | rotated) (| gates)], float32
+        if down is None:
+            down = ops.linear(x, self.w_down, out_dtype=torch.float32)
         cq = ops.latent_prepare(down, 0, s.q_rank, s.q_rank, s.kv_rank, s.rot_dim, rotary_dim, self.q_gain, self.kv_gain,
                                 s.norm_eps, cos, sin, batch.positions, batch.token_req, table, cache.data, page,
-                                write_kv=write_cache)
+                                write_kv=write_cache and s.own_kv)
         q = ops.linear(cq, self.w_uq)                                    # [tokens, heads * (head_dim + rot)]
         tokens = q.shape[0]
-        q_heads = q.view(tokens, h, s.head_dim + s.rot_dim)
-        carried = ops.head_linear(q_heads[:, :, :s.head_dim], self.w_uk, out_dtype=torch.float32)      # [heads, tokens, kv_rank]
-        queries = ops.latent_query(carried, q, h, s.head_dim, s.kv_rank, s.rot_dim, rotary_dim, cos, sin, batch.positions)
+        queries = torch.empty((tokens, h * s.row), dtype=q.dtype, device=q.device)
+        ops.head_linear(q.view(tokens, h, s.head_dim + s.rot_dim)[:, :, :s.head_dim], self.w_uk,
+                        out=queries.view(tokens, h, s.row)[:, :, :s.kv_rank])
+        ops.latent_query(queries, q, h, s.head_dim, s.kv_rank, s.rot_dim, rotary_dim, cos, sin, batch.positions)
         mixed = torch.empty((tokens, h * s.kv_rank), dtype=q.dtype, device=q.device)
         nd, dec = batch.num_decode, plan.decode
         if nd:
@@ -154,9 +184,11 @@ class LatentAttention(Mixer):
             ops.attention_prefill(queries, cache.data, table, batch.cu_seqlens, batch.prefix_lens, tile_req, tile_start,
                                   mixed, h, 1, s.row, page, s.scale, s.window, tile_rows=plan.tile_rows, dv=s.kv_rank,
                                   values_in_keys=True)
-        values = ops.head_linear(mixed.view(tokens, h, s.kv_rank), self.w_uv, out_dtype=torch.float32)  # [heads, tokens, v]
+        mixed = mixed.view(tokens, h, s.kv_rank)
         if s.out_gate:
-            out = ops.head_gate(values, down, s.q_rank + s.row, q.dtype)
+            values = ops.head_linear(mixed, self.w_uv, out_dtype=torch.float32)                         # [heads, tokens, v]
+            out = ops.head_gate(values, down, s.q_rank + (s.row if s.own_kv else 0), q.dtype)
         else:
-            out = ops.cast(values.transpose(0, 1).reshape(tokens, h * s.v_head_dim).contiguous(), q.dtype)
+            out = torch.empty((tokens, h * s.v_head_dim), dtype=q.dtype, device=q.device)
+            ops.head_linear(mixed, self.w_uv, out=out.view(tokens, h, s.v_head_dim))
         return ops.linear_auto(out, self.w_o)

@@ -90,13 +90,14 @@ class SwiGLU(FeedForward):
 @dataclass(frozen=True)
 class DenseMLPSpec:
     """The plain (ungated) feed-forward ``down(act(up(x)))``, no bias; ``activation``: "relu2" (the square of
-    max(., 0)), "gelu_tanh" or "silu"."""
+    max(., 0)), "gelu_tanh", "silu", or "xielu", which has a tensor of two learned numbers (p, q): a z^2 + z / 2 for z above
+    zero and b (e^z - 1 - z) + z / 2 below, with a = softplus(p) and b = 1/2 + softplus(q)."""
 
     hidden_size: int
     intermediate_size: int
     kind: str = "dense_mlp"
     activation: str = "relu2"
-    names: Optional[Tuple[Tuple[str, str], ...]] = None     # names of the up and down weights under the part's prefix
+    names: Optional[Tuple[Tuple[str, str], ...]] = None     # names of the up and down weights (and "act") under the part's prefix
 
     def name(self, role: str) -> str:
         return dict(self.names or ()).get(role, f"{role}_proj.weight")
@@ -107,12 +108,19 @@ class DenseMLP(FeedForward):
     def __init__(self, spec: DenseMLPSpec, prefix: str, ctx: BuildContext):
         self.spec, self.prefix, self.ctx = spec, prefix, ctx
         self.w_up = self.w_down = None
+        self.factors = (0.0, 0.0)                           # of "xielu"
 
     def tensors(self) -> Dict[str, TensorSpec]:
         h, i, p, n = self.spec.hidden_size, self.spec.intermediate_size, self.prefix, self.spec.name
-        return {f"{p}.{n('up')}": TensorSpec((i, h)), f"{p}.{n('down')}": TensorSpec((h, i))}
+        out = {f"{p}.{n('up')}": TensorSpec((i, h)), f"{p}.{n('down')}": TensorSpec((h, i))}
+        if self.spec.activation == "xielu":
+            out[f"{p}.{n('act')}"] = TensorSpec((2,), role="vector", init="zeros")
+        return out
 
     def load(self, get) -> None:
+        if self.spec.activation == "xielu":
+            a, b = torch.nn.functional.softplus(get(f"{self.prefix}.{self.spec.name('act')}").double().cpu()).tolist()
+            self.factors = (a, 0.5 + b)
         self.w_up = get(f"{self.prefix}.{self.spec.name('up')}").contiguous()
         self.w_down = get(f"{self.prefix}.{self.spec.name('down')}").contiguous()
 
@@ -120,5 +128,6 @@ class DenseMLP(FeedForward):
         ops = self.ctx.ops
         # the product with the activation in its epilogue where a kernel of that form takes the shape; else the
         # product (whole, or float32 partial sums for a few tokens) and the activation as a pass of its own
-        act = ops.linear_activation(x, self.w_up, self.spec.activation)
+        how = {"factors": self.factors} if self.spec.activation == "xielu" else {}
+        act = ops.linear_activation(x, self.w_up, self.spec.activation, **how)
         return ops.linear_auto(act, self.w_down)

@@ -35,6 +35,7 @@ class RMSNormSpec:
     suffix: str = ".weight"        # the gain's name is the part's prefix followed by this ("" where the prefix is the name)
     offset: float = 0.0            # the checkpoint stores the gain minus this (1.0: gains stored around zero); the sum
                                    # is formed once, in float32, when the gain is loaded
+    single_gain: bool = False      # the checkpoint stores one number that serves all columns (shape [])
 
 
 @register_part("norm", "rmsnorm")
@@ -44,12 +45,14 @@ class RMSNorm(Norm):
         self.weight = None
 
     def tensors(self) -> Dict[str, TensorSpec]:
-        return {f"{self.prefix}{self.spec.suffix}": TensorSpec((self.spec.size,), role="vector", init="gain")}
+        return {f"{self.prefix}{self.spec.suffix}": TensorSpec(() if self.spec.single_gain else (self.spec.size,), role="vector", init="gain")}
 
     def load(self, get) -> None:
         self.weight = get(f"{self.prefix}{self.spec.suffix}")
         if self.spec.offset:
             self.weight = (self.weight.float() + self.spec.offset).contiguous()
+        if self.spec.single_gain:
+            self.weight = self.weight.float().reshape(1).expand(self.spec.size).contiguous()      # the kernels read a gain a column
 
     def forward(self, residual, delta=None, delta_bias=None, rows=None, write_residual=True, also=None, out_dtype=None):
         """``delta`` may be a tuple of tensors to be summed; ``delta_bias`` a float32 vector added to every row;
@@ -75,3 +78,18 @@ class RMSNorm(Norm):
         outs = self.ctx.ops.add_rmsnorm_multi(residual, deltas, gains, self.spec.eps, out_dtype or self.ctx.dtype,
                                               bias=delta_bias, write_residual=write_residual)
         return outs if also is not None else outs[0]
+
+
+def enter_stream(ops, residual, delta, dtype, bias=None):
+    """Adds a pending ``delta`` (a tensor, several of them, a ``NormedDelta`` or None) and ``bias`` (a row vector) into the
+    float32 stream in place and returns the new stream itself in ``dtype``: what a sublayer takes that has no norm ahead
+    of it.  With ``dtype`` float32 that is ``residual``, which the next call changes."""
+    if isinstance(delta, NormedDelta):
+        if bias is not None:
+            raise ValueError("a normalised delta comes alone: no stream vector in the same pass")
+        return ops.add_normed(residual, delta.delta, delta.gain, delta.eps, delta.mult, dtype,
+                              **({} if delta.normalise else {"normalise": False}))
+    deltas = [d for d in delta if d is not None] if isinstance(delta, (tuple, list)) else ([delta] if delta is not None else [])
+    if deltas or bias is not None:
+        ops.add_rmsnorm_multi(residual, deltas, [], 1.0, dtype, bias=bias)
+    return ops.cast(residual, dtype)

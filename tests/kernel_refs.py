@@ -9,6 +9,7 @@ compute in float32 and round once to the output dtype.  Nothing in ``lily_b200``
 from __future__ import annotations
 
 from dataclasses import dataclass
+from typing import Optional
 
 import torch
 
@@ -475,8 +476,11 @@ def top_logprobs(logits, k):
 
 # ---- per-head products, linear attention with a data-dependent decay, attention over a latent, routed experts
 
-def head_linear(x, weight, out_dtype=None):
-    """x [tokens, heads, k], weight [heads, n, k] -> [heads, tokens, n]."""
+def head_linear(x, weight, out_dtype=None, out=None):
+    """x [tokens, heads, k], weight [heads, n, k] -> [heads, tokens, n], or into the view out [tokens, heads, n]."""
+    if out is not None:
+        out.copy_(torch.einsum("thk,hnk->thn", x.float(), weight.float()))
+        return out
     out = torch.einsum("thk,hnk->htn", x.float(), weight.float())
     return out if (out_dtype == torch.float32 or x.dtype == torch.float32) else out.to(x.dtype)
 
@@ -545,7 +549,7 @@ def _rotate_halves(t, cos, sin, positions, rotary_dim):
 
 def latent_prepare(down, q0, q_rank, kv0, rank, rot, rotary_dim, q_gain, kv_gain, eps, cos, sin, positions, token_req,
                    block_table, layer, page_size, write_kv=True):
-    x = down.float()
+    x = _sum(down).float()
     unit = lambda t: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
     cq = (unit(x[:, q0:q0 + q_rank]) * q_gain.float()).to(layer.dtype)
     if write_kv:
@@ -558,15 +562,16 @@ def latent_prepare(down, q0, q_rank, kv0, rank, rot, rotary_dim, q_gain, kv_gain
     return cq
 
 
-def latent_query(qa, q, heads, d, rank, rot, rotary_dim, cos, sin, positions):
+def latent_query(queries, q, heads, d, rank, rot, rotary_dim, cos, sin, positions):
     tokens = q.shape[0]
     turned = _rotate_halves(q.float().view(tokens, heads, d + rot)[..., d:], cos, sin, positions, rotary_dim)
-    return torch.cat([qa.float().transpose(0, 1), turned], -1).reshape(tokens, heads * (rank + rot)).to(q.dtype)
+    queries.view(tokens, heads, rank + rot)[..., rank:] = turned.to(q.dtype)
+    return queries
 
 
 def head_gate(ov, gate_rows, g0, out_dtype):
     heads, tokens, dv = ov.shape
-    g = torch.sigmoid(gate_rows[:, g0:g0 + heads].float())                      # [tokens, heads]
+    g = torch.sigmoid(_sum(gate_rows)[:, g0:g0 + heads].float())                      # [tokens, heads]
     return (ov.float().transpose(0, 1) * g[:, :, None]).reshape(tokens, heads * dv).to(out_dtype)
 
 
@@ -575,16 +580,23 @@ class ExpertRouting:
     chosen: torch.Tensor
     weights: torch.Tensor
     top: int
+    gate: Optional[torch.Tensor] = None
 
 
-def moe_route(h, router, correction, top, experts):
-    s = torch.softmax(h.float() @ router.float().t(), -1)
-    chosen = torch.topk(s + correction.float(), top, dim=-1).indices
+def moe_route(h, router, correction, top, experts, scores="softmax", renormalise=True, shared_gate=False):
+    z = h.float() @ router.float().t()
+    gate = None
+    if shared_gate:
+        z, gate = z[:, :-1], torch.sigmoid(z[:, -1])
+    s = torch.softmax(z, -1) if scores == "softmax" else torch.sigmoid(z)
+    chosen = torch.topk(s if correction is None else s + correction.float(), top, dim=-1).indices
     picked = torch.gather(s, 1, chosen)
-    return ExpertRouting(chosen.to(torch.int32), picked / (picked.sum(-1, keepdim=True) + 1e-20), top)
+    if renormalise:
+        picked = picked / (picked.sum(-1, keepdim=True) + 1e-20)
+    return ExpertRouting(chosen.to(torch.int32), picked, top, gate)
 
 
-def moe_experts(h, routing, w_gate_up, w_down, limit, alpha):
+def moe_experts(h, routing, w_gate_up, w_down, limit=0.0, alpha=0.0, activation="swish_clamped", weight_on_input=False, shared=None):
     tokens, width = h.shape
     experts = w_down.shape[0] if w_down.dim() == 3 else 0
     ff = w_down.shape[2] if experts else 0
@@ -593,12 +605,19 @@ def moe_experts(h, routing, w_gate_up, w_down, limit, alpha):
     for t in range(tokens):
         for e, a in zip(routing.chosen[t].tolist(), routing.weights[t].tolist()):
             if e < experts:
-                gu = w_gate_up[e].float() @ x[t]
-                g, u = gu[:ff].clamp(max=limit), gu[ff:].clamp(min=-limit, max=limit)
-                act = (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(h.dtype).float()
-                out[t] += a * (w_down[e].float() @ act)
+                gu = w_gate_up[e].float() @ (a * x[t] if weight_on_input else x[t])
+                g, u = gu[:ff], gu[ff:]
+                if activation == "silu":
+                    act = g * torch.sigmoid(g) * u
+                else:
+                    g, u = g.clamp(max=limit), u.clamp(min=-limit, max=limit)
+                    act = g * torch.sigmoid(alpha * g) * (u + 1.0)
+                y = w_down[e].float() @ act.to(h.dtype).float()
+                out[t] += y if weight_on_input else a * y
             else:
                 out[t] += a * x[t]
+    if shared is not None:
+        out += routing.gate[:, None] * _sum(shared).float()
     return out
 
 
@@ -623,7 +642,15 @@ def add_normed_rmsnorm(resid, delta, post_gain, post_eps, mult, weight, eps, out
     return ((v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)) * weight.float()).to(out_dtype)
 
 
-def _activate(z, activation):
+def add_normed(resid, delta, post_gain, post_eps, mult, out_dtype, normalise=True):
+    add_normed_rmsnorm(resid, delta, post_gain, post_eps, mult, None, 1.0, out_dtype, normalise=normalise)
+    return resid.to(out_dtype)
+
+
+def _activate(z, activation, factors=(0.0, 0.0)):
+    if activation == "xielu":
+        neg = z.clamp(max=0)
+        return torch.where(z > 0, factors[0] * z * z, factors[1] * (torch.expm1(neg) - neg)) + 0.5 * z
     if activation == "relu2":
         return torch.clamp(z, min=0) ** 2
     if activation == "silu":
@@ -632,12 +659,12 @@ def _activate(z, activation):
     return 0.5 * z * (1 + torch.tanh(0.7978845608028654 * (z + 0.044715 * z ** 3)))
 
 
-def activation(x, out_dtype, activation="relu2"):
-    return _activate(_sum(x).float(), activation).to(out_dtype)
+def activation(x, out_dtype, activation="relu2", factors=(0.0, 0.0)):
+    return _activate(_sum(x).float(), activation, factors).to(out_dtype)
 
 
-def linear_activation(x, weight, activation="relu2"):
-    return _activate(_sum(linear_auto(x, weight)).float(), activation).to(x.dtype)
+def linear_activation(x, weight, activation="relu2", factors=(0.0, 0.0)):
+    return _activate(_sum(linear_auto(x, weight)).float(), activation, factors).to(x.dtype)
 
 
 # ---------------------------------------------------------------------------- differential attention

@@ -237,8 +237,9 @@ def run_latent(ops, device, dtype, h, w, c, eps, page, cuts):
         cq = ops.latent_prepare(down, 0, q_rank, q_rank, rank, rot, dims, dev(w["p.dq.norm"], torch.float32),
                                 dev(w["p.dkv.norm"], torch.float32), eps, cos, sin, pos, i32([0] * n, device), table, cache, page)
         q = ops.linear(cq, w_uq)
-        carried = ops.head_linear(q.view(n, heads, d + rot)[:, :, :d], w_uk, out_dtype=torch.float32)
-        queries = ops.latent_query(carried, q, heads, d, rank, rot, dims, cos, sin, pos)
+        queries = torch.empty((n, heads * row), dtype=dtype, device=device)
+        ops.head_linear(q.view(n, heads, d + rot)[:, :, :d], w_uk, out=queries.view(n, heads, row)[:, :, :rank])
+        ops.latent_query(queries, q, heads, d, rank, rot, dims, cos, sin, pos)
         mixed = torch.empty((n, heads * rank), dtype=dtype, device=device)
         if n == 1:
             plan = ops.plan_decode_attention(dtype, 1, heads, 1, row, done + 1, dv=rank, values_in_keys=True)
