@@ -34,14 +34,14 @@
 // sets a status word (lily_attention_tc_status), the roles leave their loops and the block frees
 // its tensor memory.
 #include "common.cuh"
-
-#include <cuda.h>
+#include "tcgen05.cuh"
 
 #include <cstdlib>
-#include <mutex>
 
 namespace lily {
 namespace fa {
+
+using namespace tc5;
 
 constexpr int BQ = 128;                   // query rows per block
 constexpr int BKV = 128;                  // keys per tile
@@ -111,22 +111,6 @@ __device__ __forceinline__ float tanh_fast(float v) {
     return r;
 }
 
-__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void mbar_init(uint32_t bar, uint32_t count) {
-    asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;\n" ::"r"(bar), "r"(count));
-}
-__device__ __forceinline__ void mbar_expect_tx(uint32_t bar, uint32_t bytes) {
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void mbar_arrive(uint32_t bar) {
-    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ bool mbar_try_wait(uint32_t bar, uint32_t parity) {
-    uint32_t ok;
-    asm volatile("{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\nselp.b32 %0, 1, 0, p;\n}\n"
-                 : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-    return ok != 0;
-}
 __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatile int* abort_flag, int code) {
     for (uint32_t i = 0; i < SPIN_LIMIT; ++i) {
         if (mbar_try_wait(bar, parity)) return true;
@@ -136,90 +120,6 @@ __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatil
     atomicCAS(&g_status, 0, (code << 24) | (int)((blockIdx.x + blockIdx.y * gridDim.x) & 0xFFFFFF));
     return false;
 }
-__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, uint32_t bar, int x, int y, int z) {
-    asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];\n"
-                 ::"r"(dst), "l"(map), "r"(bar), "r"(x), "r"(y), "r"(z) : "memory");
-}
-__device__ __forceinline__ void tma_load_4d(uint32_t dst, const CUtensorMap* map, uint32_t bar, int x, int y, int z, int w) {
-    asm volatile("cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];\n"
-                 ::"r"(dst), "l"(map), "r"(bar), "r"(x), "r"(y), "r"(z), "r"(w) : "memory");
-}
-// k-major operand tile with 128-byte swizzle: rows of 128 bytes, groups of eight rows 1024 bytes apart.
-__device__ __forceinline__ uint64_t desc_k_major(uint32_t addr) {
-    uint64_t d = 0;
-    d |= (uint64_t)((addr & 0x3FFFF) >> 4);
-    d |= (uint64_t)(1024 >> 4) << 32;
-    d |= (uint64_t)1 << 46;
-    d |= (uint64_t)2 << 61;
-    return d;
-}
-// MN-major operand ([k][n] with n contiguous) with 128-byte swizzle: a row of 64 n per k, groups of
-// eight k 1024 bytes apart (stride field), the next 64 n `SUB` bytes further (leading field).
-__device__ __forceinline__ uint64_t desc_mn_major(uint32_t addr) {
-    uint64_t d = 0;
-    d |= (uint64_t)((addr & 0x3FFFF) >> 4);
-    d |= (uint64_t)(SUB >> 4) << 16;
-    d |= (uint64_t)(1024 >> 4) << 32;
-    d |= (uint64_t)1 << 46;
-    d |= (uint64_t)2 << 61;
-    return d;
-}
-__device__ __forceinline__ void umma(uint32_t tmem_c, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-    asm volatile("{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\n"
-                 "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}\n"
-                 ::"r"(tmem_c), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate) : "memory");
-}
-// The same with the A operand in tensor memory (128 lanes x k / 2 columns of bfloat16 pairs).
-__device__ __forceinline__ void umma_ts(uint32_t tmem_c, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-    asm volatile("{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\n"
-                 "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}\n"
-                 ::"r"(tmem_c), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate) : "memory");
-}
-__device__ __forceinline__ void umma_commit(uint32_t bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n" ::"r"(bar) : "memory");
-}
-// 32 consecutive columns of this thread's lane of tensor memory; follow with tmem_wait_ld().
-__device__ __forceinline__ void tmem_ld32(uint32_t taddr, float* r) {
-    uint32_t* u = reinterpret_cast<uint32_t*>(r);
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-                 "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];\n"
-                 : "=r"(u[0]), "=r"(u[1]), "=r"(u[2]), "=r"(u[3]), "=r"(u[4]), "=r"(u[5]), "=r"(u[6]), "=r"(u[7]),
-                   "=r"(u[8]), "=r"(u[9]), "=r"(u[10]), "=r"(u[11]), "=r"(u[12]), "=r"(u[13]), "=r"(u[14]), "=r"(u[15]),
-                   "=r"(u[16]), "=r"(u[17]), "=r"(u[18]), "=r"(u[19]), "=r"(u[20]), "=r"(u[21]), "=r"(u[22]), "=r"(u[23]),
-                   "=r"(u[24]), "=r"(u[25]), "=r"(u[26]), "=r"(u[27]), "=r"(u[28]), "=r"(u[29]), "=r"(u[30]), "=r"(u[31])
-                 : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_wait_ld() { asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory"); }
-__device__ __forceinline__ void tmem_st32(uint32_t taddr, const float* r) {
-    const uint32_t* u = reinterpret_cast<const uint32_t*>(r);
-    asm volatile("tcgen05.st.sync.aligned.32x32b.x32.b32 [%32], "
-                 "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31};\n"
-                 ::"r"(u[0]), "r"(u[1]), "r"(u[2]), "r"(u[3]), "r"(u[4]), "r"(u[5]), "r"(u[6]), "r"(u[7]),
-                   "r"(u[8]), "r"(u[9]), "r"(u[10]), "r"(u[11]), "r"(u[12]), "r"(u[13]), "r"(u[14]), "r"(u[15]),
-                   "r"(u[16]), "r"(u[17]), "r"(u[18]), "r"(u[19]), "r"(u[20]), "r"(u[21]), "r"(u[22]), "r"(u[23]),
-                   "r"(u[24]), "r"(u[25]), "r"(u[26]), "r"(u[27]), "r"(u[28]), "r"(u[29]), "r"(u[30]), "r"(u[31]),
-                   "r"(taddr) : "memory");
-}
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const float* r) {
-    const uint32_t* u = reinterpret_cast<const uint32_t*>(r);
-    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15};\n"
-                 ::"r"(u[0]), "r"(u[1]), "r"(u[2]), "r"(u[3]), "r"(u[4]), "r"(u[5]), "r"(u[6]), "r"(u[7]),
-                   "r"(u[8]), "r"(u[9]), "r"(u[10]), "r"(u[11]), "r"(u[12]), "r"(u[13]), "r"(u[14]), "r"(u[15]),
-                   "r"(taddr) : "memory");
-}
-__device__ __forceinline__ void tmem_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory"); }
-__device__ __forceinline__ float ex2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ uint32_t pack2(float a, float b) {
-    __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<uint32_t*>(&v);
-}
-
 template <int D>
 __global__ void __launch_bounds__(THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const Params p) {
@@ -374,7 +274,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (ok) { FA_TIC(); ok = mbar_wait(v_full + 8 * s, (uint32_t)((j / STAGES) & 1), abort_flag, 6); FA_TOC(3, true); }
                 if (!ok) break;
                 tc_fence_after();
-                const uint64_t dv = desc_mn_major(v_smem + s * TILE), dp = desc_k_major(p_smem + b * P_TILE);
+                const uint64_t dv = desc_mn_major(v_smem + s * TILE, SUB), dp = desc_k_major(p_smem + b * P_TILE);
 #pragma unroll
                 for (int kk = 0; kk < BKV / 16; ++kk) {
                     const uint64_t db = dv + (uint64_t)(kk * 2048 >> 4);
@@ -734,7 +634,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 ok = mbar_wait(v_full, 0, abort_flag, 6);
                 tc_fence_after();
                 uint32_t phase = 0;
-                const uint64_t dq = desc_k_major(q_smem), dk = desc_k_major(k_smem), dv = desc_mn_major(v_smem);
+                const uint64_t dq = desc_k_major(q_smem), dk = desc_k_major(k_smem), dv = desc_mn_major(v_smem, SUB);
                 for (int kind = 0; kind < 4 && ok; ++kind) {
                     FA_TIC();
                     const int reps = kind == 0 ? 4 : (kind == 3 ? 0 : (kind == 1 ? 1 : 4));
@@ -765,7 +665,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
                     { FA_TIC(); ok = mbar_wait(p_full + 8 * h, (uint32_t)(j & 1), abort_flag, 5); FA_TOC(4 + h, true); }
                     if (!ok) break;
                     tc_fence_after();
-                    const uint64_t dv = desc_mn_major(v_smem + s * TILE);
+                    const uint64_t dv = desc_mn_major(v_smem + s * TILE, SUB);
 #pragma unroll
                     for (int kk = 0; kk < BKV / 16; ++kk)
                         umma_ts(tmem_o + (uint32_t)(h * D), tmem + (uint32_t)(h * BKV + kk * 8), dv + (uint64_t)(kk * 2048 >> 4), idesc_o,
@@ -914,23 +814,6 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
 
 // ---- host side --------------------------------------------------------------------------------
 
-typedef CUresult (*EncodeTiled)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-static EncodeTiled encoder() {
-    static EncodeTiled fn = nullptr;
-    static std::once_flag once;
-    std::call_once(once, [] {
-        void* ptr = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) == cudaSuccess &&
-            q == cudaDriverEntryPointSuccess)
-            fn = (EncodeTiled)ptr;
-    });
-    return fn;
-}
-
 // Launches the kernel of head size D with one head or two heads a block (the shared memory limits are raised once).
 template <int D>
 static int launch(bool two, int nq, int tiles, cudaStream_t stream, const CUtensorMap& map_q, const CUtensorMap& map_kv, const Params& p) {
@@ -999,7 +882,7 @@ LILY_API int lily_attention_prefill_tc(const void* q, const void* kv, void* out,
     LILY_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention_prefill_tc: %d query heads over %d kv heads", nq, nkv);
     LILY_REQUIRE(tiles <= 65535 && tokens > 0 && num_pages > 0, "attention_prefill_tc: tiles=%d tokens=%d pages=%d", tiles, tokens, num_pages);
     LILY_REQUIRE(((uintptr_t)q % 16 == 0) && ((uintptr_t)kv % 16 == 0) && ((uintptr_t)out % 16 == 0), "attention_prefill_tc: operands must be 16-byte aligned");
-    fa::EncodeTiled enc = fa::encoder();
+    tc5::EncodeTiled enc = tc5::encoder();
     LILY_REQUIRE(enc != nullptr, "attention_prefill_tc: the driver does not offer cuTensorMapEncodeTiled");
     CUtensorMap map_q, map_kv;
     {

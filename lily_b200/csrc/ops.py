@@ -60,6 +60,7 @@ _SIGNATURES = {
     "lily_ssd_combine": [_vp, _sz, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "lily_gated_group_rmsnorm": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _f, _i, _vp],
     "lily_latent_attention_prefill_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
+    "lily_latent_attention_prefill_tc": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp],
     "lily_latent_attention_decode_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
     "lily_add_rmsnorm_multi": [_vp, _vp, _i, _i, _sz, _vp, _i, _i, _sz, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _i, _vp],
     "lily_gemm_fp32_heads": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _sz, _sz, _sz, _vp],
@@ -124,6 +125,11 @@ def library():
         lib.lily_latent_attention_mma_tile_tokens.argtypes = [_i]
         lib.lily_latent_attention_mma_tile_tokens.restype = _i
         lib.lily_latent_attention_status.restype = _i
+        lib.lily_latent_attention_tc_takes.argtypes = [_i, _i, _i]
+        lib.lily_latent_attention_tc_takes.restype = _i
+        lib.lily_latent_attention_tc_tile_tokens.argtypes = [_i]
+        lib.lily_latent_attention_tc_tile_tokens.restype = _i
+        lib.lily_latent_attention_tc_status.restype = _i
         lib.lily_moe_tile_rows.restype = _i
         lib.lily_delta_rule_max_head_dim.restype = _i
         lib.lily_selective_scan_max_state.restype = _i
@@ -570,7 +576,11 @@ def uses_tcgen05_attention(dtype: torch.dtype, d: int, page_size: int, new_token
             and bool(library().lily_attention_prefill_tc_takes(int(d), int(page_size))))
 
 
+# LILY_B200_LATENT_ATTENTION=simt keeps attention over a cached latent on the CUDA cores, =mma its prompt portions on mma.sync
 _SIMT_LATENT = os.environ.get("LILY_B200_LATENT_ATTENTION", "") == "simt"
+_TC_LATENT = os.environ.get("LILY_B200_LATENT_ATTENTION", "") not in ("simt", "mma")
+# A step whose portions bring fewer (token, head) rows than this runs them through the mma.sync kernel (blocks of 32 rows)
+LATENT_TC_MIN_ROWS = 2048
 
 
 def latent_tensor_cores(dtype: torch.dtype, d: int, dv: Optional[int], nkv: int = 1, softcap: Optional[float] = None) -> bool:
@@ -580,10 +590,17 @@ def latent_tensor_cores(dtype: torch.dtype, d: int, dv: Optional[int], nkv: int 
             and bool(library().lily_latent_attention_mma_takes(int(d), int(dv))))
 
 
+def latent_tcgen05(dtype: torch.dtype, d: int, dv: Optional[int], page_size: int, nkv: int = 1, softcap: Optional[float] = None) -> bool:
+    """Whether the tcgen05 kernel for prompt portions over cached latents takes these sizes (rows and values of whole 16-byte
+    pieces, rows of up to 640 numbers, pages of a multiple of 64 positions)."""
+    return (_TC_LATENT and latent_tensor_cores(dtype, d, dv, nkv, softcap)
+            and bool(library().lily_latent_attention_tc_takes(int(d), int(dv), int(page_size))))
+
+
 def latent_attention_status() -> int:
-    """0, or 1 + the block of the first bounded wait for a key tile that gave up in the tensor-core kernel for cached
-    latents (synchronises; the word is cleared when read)."""
-    return int(library().lily_latent_attention_status())
+    """0, or a code of the first bounded wait that gave up in a tensor-core kernel for cached latents: 1 + the block from the
+    mma.sync kernel, a number from 2^24 on from the tcgen05 kernel (synchronises; the words are cleared when read)."""
+    return int(library().lily_latent_attention_status()) or int(library().lily_latent_attention_tc_status())
 
 
 def prefill_tile_rows(dtype: torch.dtype = torch.float32, d: int = 0, page_size: int = 0, new_tokens: int = 0,
@@ -593,7 +610,10 @@ def prefill_tile_rows(dtype: torch.dtype = torch.float32, d: int = 0, page_size:
     where it differs), page size, number of new tokens and kind of scores and mask."""
     lib = library()
     if values_in_keys and heads and latent_tensor_cores(dtype, d, dv, softcap=softcap):
-        return int(lib.lily_latent_attention_mma_tile_tokens(int(heads)))
+        few = int(lib.lily_latent_attention_mma_tile_tokens(int(heads)))
+        many = int(lib.lily_latent_attention_tc_tile_tokens(int(heads)))
+        # a tile height names its kernel; where both kernels' tiles hold one token (65 heads and more) it is the tcgen05 one
+        return many if latent_tcgen05(dtype, d, dv, page_size) and (many == few or new_tokens * heads >= LATENT_TC_MIN_ROWS) else few
     if (sink or all_values) and sink_on_tensor_cores(dtype, d, dv, values_in_keys, softcap):
         return int(lib.lily_attention_prefill_mma_rows())
     if sink or all_values:
@@ -661,6 +681,13 @@ def attention_prefill(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torc
     lib = library()
     dv = int(dv or d)
     cap = float(softcap or 0.0)
+    if (values_in_keys and latent_tcgen05(q.dtype, d, dv, page_size, nkv, softcap)
+            and tile_rows == int(lib.lily_latent_attention_tc_tile_tokens(int(nq)))):
+        _call("lily_latent_attention_prefill_tc", _p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"),
+              block_table.shape[-1], _i32(cu_seqlens, "cu_seqlens"), _i32(prefix_lens, "prefix_lens"),
+              _i32(tile_req, "tile_req"), _i32(tile_start, "tile_start"), tile_req.numel(), int(tile_rows), nq, d, dv,
+              page_size, int(window or 0), float(scale), q.shape[0], kv_layer.shape[0], _stream())
+        return
     if (values_in_keys and latent_tensor_cores(q.dtype, d, dv, nkv, softcap)
             and tile_rows == int(lib.lily_latent_attention_mma_tile_tokens(int(nq)))):
         _call("lily_latent_attention_prefill_mma", _p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"),
