@@ -169,7 +169,7 @@ def kernel_table(z: dict, tokens: int, batch: int, context: int, reps: int = 30,
         q = (rnd(batch, h_ * row) / 8).to(dt)
         out = torch.empty((batch, h_ * rank), device=dev, dtype=dt)
         seq = torch.full((batch,), context, device=dev, dtype=torch.int32)
-        plan = ops.plan_decode_attention(dt, batch, h_, 1, row, seen, dv=rank, values_in_keys=True)
+        plan = ops.plan_decode_attention(dt, batch, h_, 1, row, seen, dv=rank, values_in_keys=True, page_size=page)
         scratch = torch.empty(max(1, plan.scratch_floats), device=dev)
         fns.append(lambda q=q, cache=cache, table=table, out=out, seq=seq, scratch=scratch, plan=plan: ops.attention_decode(
             q, cache, table, seq, out, scratch, plan.splits, h_, 1, row, page, la["scale"], window, dv=rank, values_in_keys=True))

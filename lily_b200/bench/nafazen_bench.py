@@ -177,7 +177,7 @@ def kernel_table(z: dict, tokens: int, batch: int, context: int, reps: int = 30,
         seq = torch.full((batch,), context, device=dev, dtype=torch.int32)
         cache, q = rnd(batch * pages + 1, page * row).to(dt), (rnd(batch, heads * row) / 8).to(dt)
         out = torch.empty((batch, heads * rank), device=dev, dtype=dt)
-        plan = ops.plan_decode_attention(dt, batch, heads, 1, row, context, dv=rank, values_in_keys=True)
+        plan = ops.plan_decode_attention(dt, batch, heads, 1, row, context, dv=rank, values_in_keys=True, page_size=page)
         scratch = torch.empty(max(1, plan.scratch_floats), device=dev)
         fns.append(lambda q=q, cache=cache, table=table, out=out, seq=seq, scratch=scratch, plan=plan: ops.attention_decode(
             q, cache, table, seq, out, scratch, plan.splits, heads, 1, row, page, att["scale"], None, dv=rank, values_in_keys=True))

@@ -1,4 +1,4 @@
-// Prefill attention over a cached latent on the fifth-generation tensor cores (bfloat16): all query heads share one cached
+// Attention over a cached latent on the fifth-generation tensor cores (bfloat16): all query heads share one cached
 // row per position, [latent (rank) | rotated key part], and the values are the first `rank` columns of the same rows.
 //
 // The query rows of a request are its (token, head) pairs in that order, which is how they lie in memory.  A block takes
@@ -17,6 +17,11 @@
 //   warps 2-5  one thread a query row, which holds the row's 128 scores in registers: maximum, then P = exp2(s * scale -
 //            max) as bfloat16 pairs over the S columns it came from, running maximum and sum in float32.  The maximum that P is taken against moves only when the true one is 2^8 ahead (O is rescaled in
 //            tensor memory then).  At the end O is divided by the sum and stored.
+//
+// Decode is the same kernel with one new token a request at position seq_len - 1: a tile is one token's heads, and the keys
+// may be cut into ranges of whole tiles whose (max, sum, output) go to scratch in the layout the combine kernel merges
+// (lily_attention_combine: [requests, heads, ranges, rank] outputs, then [.., 2]).  Fewer than 128 heads leave rows of
+// the products unused (their time is the tensor cores' for 128 rows whatever the heads).
 //
 // Keys past the last one a block sees and rows past the tile's are computed on whatever the pages and the neighbouring
 // query rows hold (finite everywhere) and masked, or not stored.  Every wait is bounded; one that runs out sets a status
@@ -51,11 +56,15 @@ struct Params {
     const int* prefix_lens;
     const int* tile_req;
     const int* tile_start;
+    const int* seq_lens;                  // decode: [requests]; null: prompt portions
+    float* part_o;                        // decode with key ranges
+    float* part_ml;
+    int splits;
     __nv_bfloat16* out;                   // [tokens, heads, rank]
     int bt_stride, tiles, tile_tokens, row_blocks, heads, row, rank, page_size, window;
     int chunks;                           // pieces of 64 columns of a row
     int col_blocks, cols;                 // column blocks and value columns of one (a multiple of 16)
-    int stages;
+    int stages, q_rows;                   // rows of the queries' box
     float scale_log2;
 };
 
@@ -125,26 +134,45 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
     pdl_wait();
     pdl_launch_dependents();
 
-    const int cb = blockIdx.x % p.col_blocks, work = blockIdx.x / p.col_blocks;
+    const int cb = blockIdx.x % p.col_blocks;
+    int work = blockIdx.x / p.col_blocks;
     const int row0 = (work % p.row_blocks) * BQ;                    // this block's first row of the tile's
-    const int tile = p.tiles - 1 - work / p.row_blocks;             // the last tiles, which see the most keys, go first
-    const int req = uniform(p.tile_req[tile]), start = uniform(p.tile_start[tile]);
-    const int tok0 = uniform(p.cu_seqlens[req]) + start;
-    const int ntok = min(p.tile_tokens, uniform(p.cu_seqlens[req + 1]) - tok0);
+    work /= p.row_blocks;
+    const bool decode = p.seq_lens != nullptr;
+    int req, tok0, ntok, pos0, range = 0;
+    if (decode) {
+        range = work % p.splits;
+        req = work / p.splits;
+        tok0 = req;
+        ntok = 1;
+        pos0 = uniform(p.seq_lens[req]) - 1;
+    } else {
+        const int tile = p.tiles - 1 - work;                        // the last tiles, which see the most keys, go first
+        req = uniform(p.tile_req[tile]);
+        const int start = uniform(p.tile_start[tile]);
+        tok0 = uniform(p.cu_seqlens[req]) + start;
+        ntok = min(p.tile_tokens, uniform(p.cu_seqlens[req + 1]) - tok0);
+        pos0 = uniform(p.prefix_lens[req]) + start;                 // position of the tile's first token
+    }
     const int nrows = ntok * p.heads;
     const int rows_valid = min(BQ, nrows - row0);                   // >= 1: a tile of several tokens has one row block
-    const int pos0 = uniform(p.prefix_lens[req]) + start;                    // position of the tile's first token
     const int first_pos = pos0 + row0 / p.heads, last_pos = pos0 + (row0 + rows_valid - 1) / p.heads;
-    const int kv_end = last_pos + 1;
+    int kv_end = last_pos + 1;
     const int k_lo = (p.window > 0 && first_pos + 1 > p.window) ? first_pos + 1 - p.window : 0;
-    const int jt0 = k_lo / BKV;
-    const int n = (kv_end - 1) / BKV - jt0 + 1;                     // key tiles of this block (>= 1)
+    int jt0 = k_lo / BKV;
+    int n = (kv_end - 1) / BKV - jt0 + 1;                           // key tiles of this block (>= 1, but for a range past the keys)
+    if (decode && p.splits > 1) {
+        const int per = (n + p.splits - 1) / p.splits;
+        jt0 += range * per;
+        n = min(per, n - range * per);
+        kv_end = min(kv_end, (jt0 + per) * BKV);
+    }
     const int v0 = cb * p.cols, nv = (p.cols + 63) / 64;            // first value column, boxes of 64 columns
 
     if (warp == 0) {
         const int* table = p.block_table + (size_t)req * p.bt_stride;
         if (elect_one()) {
-            mbar_expect_tx(q_full, NC * STAGE);
+            mbar_expect_tx(q_full, NC * p.q_rows * 128);
             for (int c = 0; c < NC; ++c) tma_load_2d(q_smem + c * STAGE, &map_q, q_full, c * 64, tok0 * p.heads + row0);
         }
         int it = 0, s = 0;                                          // pieces issued so far; the next one's stage
@@ -177,7 +205,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
                 next();
             }
         };
-        keys(0);
+        if (n > 0) keys(0);
         for (int j = 0; j < n && ok; ++j) {
             if (j + 1 < n) {
                 keys(j + 1);
@@ -238,7 +266,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
             }
             return true;
         };
-        if (ok) ok = scores(0);
+        if (ok && n > 0) ok = scores(0);
         for (int j = 0; j < n && ok; ++j) {
             const int b = j & 1;
             if (j + 1 < n) {
@@ -270,6 +298,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
         const int pos = pos0 + (row0 + row) / p.heads;
         const uint32_t my_o = tmem_o + lane_addr;
         const int pieces = (p.cols + 31) / 32;
+        const bool idle = (warp & 3) * 32 >= rows_valid;
         float m_used = -INFINITY, l = 0.f;
         bool ok = true;
         for (int j = 0; j < n && ok; ++j) {
@@ -277,6 +306,10 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
             const uint32_t my_s = tmem + lane_addr + (uint32_t)(b * BKV);
             ok = mbar_wait(s_full + 8 * b, (uint32_t)((j >> 1) & 1), abort_flag, 7);
             if (!ok) break;
+            if (idle) {                                             // none of this warp's rows is stored: whatever P they have will do
+                mbar_arrive(p_full + 8 * b);
+                continue;
+            }
             tc_fence_after();
             const int kb = (jt0 + j) * BKV;
             const bool need_mask = kb + BKV - 1 > first_pos || (p.window > 0 && kb <= last_pos - p.window);
@@ -336,25 +369,42 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
             tc_fence_before();
             mbar_arrive(p_full + 8 * b);
         }
-        if (ok) ok = mbar_wait(pv_done + 8 * ((n - 1) & 1), (uint32_t)(((n - 1) >> 1) & 1), abort_flag, 10);
-        if (ok) {
+        if (ok && n > 0) ok = mbar_wait(pv_done + 8 * ((n - 1) & 1), (uint32_t)(((n - 1) >> 1) & 1), abort_flag, 10);
+        if (ok && !idle) {
             tc_fence_after();
-            const float inv = l > 0.f ? 1.f / l : 0.f;
+            const bool partial = decode && p.splits > 1;
+            const float inv = partial ? 1.f : (l > 0.f ? 1.f / l : 0.f);
             const int last = min(p.rank, v0 + p.cols);              // the rank is a multiple of 8: an eighth is in or out as a whole
-            __nv_bfloat16* dst = p.out + ((size_t)tok0 * p.heads + row0 + row) * p.rank;
+            const size_t line = (size_t)tok0 * p.heads + row0 + row, slot = line * p.splits + range;
+            __nv_bfloat16* dst = p.out + line * p.rank;
+            float* dst_f = p.part_o + slot * p.rank;
+            if (partial && cb == 0 && row < rows_valid) {
+                p.part_ml[slot * 2] = m_used * (p.scale_log2 * 0.6931471805599453f);      // natural units of the scaled score
+                p.part_ml[slot * 2 + 1] = l;
+            }
 #pragma unroll 1
             for (int c = 0; c < pieces; ++c) {
                 float o[32];
-                tmem_ld32(my_o + (uint32_t)(c * 32), o);
-                tmem_wait_ld();
+                if (n > 0) {
+                    tmem_ld32(my_o + (uint32_t)(c * 32), o);
+                    tmem_wait_ld();
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 32; ++e) o[e] = 0.f;        // a range without keys
+                }
                 if (row < rows_valid) {
 #pragma unroll
                     for (int v = 0; v < 4; ++v) {
                         const int col = v0 + c * 32 + v * 8;
-                        if (col < last)
+                        if (col >= last) continue;
+                        if (partial) {
+                            *reinterpret_cast<float4*>(dst_f + col) = make_float4(o[v * 8], o[v * 8 + 1], o[v * 8 + 2], o[v * 8 + 3]);
+                            *reinterpret_cast<float4*>(dst_f + col + 4) = make_float4(o[v * 8 + 4], o[v * 8 + 5], o[v * 8 + 6], o[v * 8 + 7]);
+                        } else {
                             *reinterpret_cast<uint4*>(dst + col) =
                                 make_uint4(pack2(o[v * 8] * inv, o[v * 8 + 1] * inv), pack2(o[v * 8 + 2] * inv, o[v * 8 + 3] * inv),
                                            pack2(o[v * 8 + 4] * inv, o[v * 8 + 5] * inv), pack2(o[v * 8 + 6] * inv, o[v * 8 + 7] * inv));
+                        }
                     }
                 }
             }
@@ -396,50 +446,83 @@ LILY_API int lily_latent_attention_tc_takes(int row, int rank, int page_size) {
 // New tokens a tile holds for this many heads (a block takes 128 of the tile's (token, head) rows).
 LILY_API int lily_latent_attention_tc_tile_tokens(int heads) { return heads >= lt::BQ ? 1 : lt::BQ / heads; }
 
+// Column blocks the values of this rank are cut into (each forms the scores for itself).
+LILY_API int lily_latent_attention_tc_col_blocks(int rank) { return (rank + lt::MAX_COLUMNS - 1) / lt::MAX_COLUMNS; }
+
+namespace lily {
+namespace lt {
+
+// Fills in what both entries share, encodes the tensor maps and launches `units` (tile or request and range) blocks a row and column block.
+static int launch(Params& p, long units, const void* q, const void* cache, int tokens, int num_pages, float scale, cudaStream_t stream) {
+    LILY_REQUIRE(lily_latent_attention_tc_takes(p.row, p.rank, p.page_size), "latent_attention_tc: rows of %d with rank %d in pages of %d are not for this kernel", p.row, p.rank, p.page_size);
+    LILY_REQUIRE(p.heads > 0 && tokens > 0 && num_pages > 0 && scale > 0.f, "latent_attention_tc: heads=%d tokens=%d pages=%d scale=%g", p.heads, tokens, num_pages, scale);
+    LILY_REQUIRE(((uintptr_t)q % 16 == 0) && ((uintptr_t)cache % 16 == 0) && ((uintptr_t)p.out % 16 == 0) && ((uintptr_t)p.part_o % 16 == 0),
+                 "latent_attention_tc: operands must be 16-byte aligned");
+    const int tile_rows = p.tile_tokens * p.heads;
+    p.row_blocks = (tile_rows + BQ - 1) / BQ;
+    p.chunks = (p.row + 63) / 64;
+    p.col_blocks = lily_latent_attention_tc_col_blocks(p.rank);
+    p.cols = ((p.rank + p.col_blocks - 1) / p.col_blocks + 15) / 16 * 16;
+    p.stages = ring_stages(p.row);
+    p.q_rows = tile_rows >= BQ ? BQ : (tile_rows + 7) / 8 * 8;      // rows of a tile past its last are computed on whatever is there
+    p.scale_log2 = scale * 1.4426950408889634f;
+    CUtensorMap map_q, map_k, map_v;
+    {
+        const cuuint64_t dims[2] = {(cuuint64_t)p.row, (cuuint64_t)tokens * p.heads}, strides[1] = {(cuuint64_t)p.row * 2};
+        const cuuint32_t box[2] = {64, (cuuint32_t)p.q_rows};
+        LILY_REQUIRE(encode(&map_q, q, 2, dims, strides, box), "latent_attention_tc: the tensor map of the queries was refused");
+    }
+    {
+        const cuuint64_t dims[3] = {(cuuint64_t)p.row, (cuuint64_t)p.page_size, (cuuint64_t)num_pages};
+        const cuuint64_t strides[2] = {(cuuint64_t)p.row * 2, (cuuint64_t)p.page_size * p.row * 2};
+        const cuuint32_t box_k[3] = {64, 64, 1}, box_v[3] = {64, (cuuint32_t)VKEYS, 1};
+        LILY_REQUIRE(encode(&map_k, cache, 3, dims, strides, box_k) && encode(&map_v, cache, 3, dims, strides, box_v),
+                     "latent_attention_tc: the tensor map of the cache was refused");
+    }
+    const size_t smem = (size_t)(p.chunks + p.stages) * STAGE + TAIL;
+    static size_t granted = 0;
+    if (smem > granted) {
+        cudaError_t e = cudaFuncSetAttribute(latent_attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) { set_error("latent_attention_tc: cannot get %zu bytes of shared memory: %s", smem, cudaGetErrorString(e)); return 2; }
+        granted = smem;
+    }
+    const long blocks = units * p.row_blocks * p.col_blocks;
+    LILY_REQUIRE(blocks < (1l << 31), "latent_attention_tc: %ld blocks", blocks);
+    launch_pdl(latent_attention_tc_kernel, dim3((unsigned)blocks), dim3(THREADS), smem, stream, map_q, map_k, map_v, p);
+    LILY_CHECK_LAUNCH("latent_attention_tc");
+    return 0;
+}
+
+}  // namespace lt
+}  // namespace lily
+
+// Prompt portions: `tiles` of `tile_tokens` new tokens (request and offset); q and out have `tokens` rows in all.
 LILY_API int lily_latent_attention_prefill_tc(const void* q, const void* cache, void* out, const int* block_table, int bt_stride,
                                               const int* cu_seqlens, const int* prefix_lens, const int* tile_req, const int* tile_start,
                                               int tiles, int tile_tokens, int heads, int row, int rank, int page_size, int window,
                                               float scale, int tokens, int num_pages, cudaStream_t stream) {
     if (tiles == 0) return 0;
-    LILY_REQUIRE(lily_latent_attention_tc_takes(row, rank, page_size), "latent_attention_tc: rows of %d with rank %d in pages of %d are not for this kernel", row, rank, page_size);
-    LILY_REQUIRE(heads > 0 && tile_tokens > 0 && (tile_tokens == 1 || tile_tokens * heads <= lt::BQ), "latent_attention_tc: tiles of %d tokens of %d heads", tile_tokens, heads);
-    LILY_REQUIRE(tokens > 0 && num_pages > 0 && scale > 0.f, "latent_attention_tc: tokens=%d pages=%d scale=%g", tokens, num_pages, scale);
-    LILY_REQUIRE(((uintptr_t)q % 16 == 0) && ((uintptr_t)cache % 16 == 0) && ((uintptr_t)out % 16 == 0), "latent_attention_tc: operands must be 16-byte aligned");
-    CUtensorMap map_q, map_k, map_v;
-    {
-        const cuuint64_t dims[2] = {(cuuint64_t)row, (cuuint64_t)tokens * heads}, strides[1] = {(cuuint64_t)row * 2};
-        const cuuint32_t box[2] = {64, (cuuint32_t)lt::BQ};
-        LILY_REQUIRE(lt::encode(&map_q, q, 2, dims, strides, box), "latent_attention_tc: the tensor map of the queries was refused");
-    }
-    {
-        const cuuint64_t dims[3] = {(cuuint64_t)row, (cuuint64_t)page_size, (cuuint64_t)num_pages};
-        const cuuint64_t strides[2] = {(cuuint64_t)row * 2, (cuuint64_t)page_size * row * 2};
-        const cuuint32_t box_k[3] = {64, 64, 1}, box_v[3] = {64, (cuuint32_t)lt::VKEYS, 1};
-        LILY_REQUIRE(lt::encode(&map_k, cache, 3, dims, strides, box_k) && lt::encode(&map_v, cache, 3, dims, strides, box_v),
-                     "latent_attention_tc: the tensor map of the cache was refused");
-    }
+    LILY_REQUIRE(tile_tokens > 0 && (tile_tokens == 1 || tile_tokens * heads <= lt::BQ), "latent_attention_tc: tiles of %d tokens of %d heads", tile_tokens, heads);
     lt::Params p{};
     p.block_table = block_table; p.cu_seqlens = cu_seqlens; p.prefix_lens = prefix_lens; p.tile_req = tile_req; p.tile_start = tile_start;
     p.out = (__nv_bfloat16*)out; p.bt_stride = bt_stride; p.tiles = tiles; p.tile_tokens = tile_tokens; p.heads = heads; p.row = row;
-    p.rank = rank; p.page_size = page_size; p.window = window;
-    p.row_blocks = (tile_tokens * heads + lt::BQ - 1) / lt::BQ;
-    p.chunks = (row + 63) / 64;
-    p.col_blocks = (rank + lt::MAX_COLUMNS - 1) / lt::MAX_COLUMNS;
-    p.cols = ((rank + p.col_blocks - 1) / p.col_blocks + 15) / 16 * 16;
-    p.stages = lt::ring_stages(row);
-    p.scale_log2 = scale * 1.4426950408889634f;
-    const size_t smem = (size_t)(p.chunks + p.stages) * lt::STAGE + lt::TAIL;
-    static size_t granted = 0;
-    if (smem > granted) {
-        cudaError_t e = cudaFuncSetAttribute(lt::latent_attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) { set_error("latent_attention_tc: cannot get %zu bytes of shared memory: %s", smem, cudaGetErrorString(e)); return 2; }
-        granted = smem;
-    }
-    const long blocks = (long)tiles * p.row_blocks * p.col_blocks;
-    LILY_REQUIRE(blocks < (1l << 31), "latent_attention_tc: %ld blocks", blocks);
-    launch_pdl(lt::latent_attention_tc_kernel, dim3((unsigned)blocks), dim3(lt::THREADS), smem, stream, map_q, map_k, map_v, p);
-    LILY_CHECK_LAUNCH("latent_attention_tc");
-    return 0;
+    p.rank = rank; p.page_size = page_size; p.window = window; p.splits = 1;
+    return lt::launch(p, tiles, q, cache, tokens, num_pages, scale, stream);
+}
+
+// One new token a request: q [requests, heads, row], out [requests, heads, rank]; with more than one key range the ranges'
+// results go to scratch, ahead of lily_attention_combine.
+LILY_API int lily_latent_attention_decode_tc(const void* q, const void* cache, void* out, const int* block_table, int bt_stride,
+                                             const int* seq_lens, float* scratch, int requests, int splits, int heads, int row, int rank,
+                                             int page_size, int window, float scale, int num_pages, cudaStream_t stream) {
+    if (requests == 0) return 0;
+    LILY_REQUIRE(seq_lens && splits >= 1 && (splits == 1 || scratch), "latent_attention_tc: %d key ranges need scratch", splits);
+    lt::Params p{};
+    p.block_table = block_table; p.seq_lens = seq_lens; p.splits = splits; p.out = (__nv_bfloat16*)out; p.bt_stride = bt_stride;
+    p.tiles = requests; p.tile_tokens = 1; p.heads = heads; p.row = row; p.rank = rank; p.page_size = page_size; p.window = window;
+    p.part_o = splits > 1 ? scratch : nullptr;
+    p.part_ml = splits > 1 ? scratch + (size_t)requests * heads * splits * rank : nullptr;
+    return lt::launch(p, (long)requests * splits, q, cache, requests, num_pages, scale, stream);
 }
 
 // 0 while no wait has given up since the last call; else (code << 24 | block).  Codes: 1, 2 the loader waiting for a free

@@ -61,6 +61,7 @@ _SIGNATURES = {
     "lily_gated_group_rmsnorm": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _f, _i, _vp],
     "lily_latent_attention_prefill_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
     "lily_latent_attention_prefill_tc": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp],
+    "lily_latent_attention_decode_tc": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
     "lily_latent_attention_decode_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
     "lily_add_rmsnorm_multi": [_vp, _vp, _i, _i, _sz, _vp, _i, _i, _sz, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _i, _vp],
     "lily_gemm_fp32_heads": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _sz, _sz, _sz, _vp],
@@ -130,6 +131,8 @@ def library():
         lib.lily_latent_attention_tc_tile_tokens.argtypes = [_i]
         lib.lily_latent_attention_tc_tile_tokens.restype = _i
         lib.lily_latent_attention_tc_status.restype = _i
+        lib.lily_latent_attention_tc_col_blocks.argtypes = [_i]
+        lib.lily_latent_attention_tc_col_blocks.restype = _i
         lib.lily_moe_tile_rows.restype = _i
         lib.lily_delta_rule_max_head_dim.restype = _i
         lib.lily_selective_scan_max_state.restype = _i
@@ -576,11 +579,11 @@ def uses_tcgen05_attention(dtype: torch.dtype, d: int, page_size: int, new_token
             and bool(library().lily_attention_prefill_tc_takes(int(d), int(page_size))))
 
 
-# LILY_B200_LATENT_ATTENTION=simt keeps attention over a cached latent on the CUDA cores, =mma its prompt portions on mma.sync
+# LILY_B200_LATENT_ATTENTION=simt keeps attention over a cached latent on the CUDA cores, =mma on mma.sync
 _SIMT_LATENT = os.environ.get("LILY_B200_LATENT_ATTENTION", "") == "simt"
 _TC_LATENT = os.environ.get("LILY_B200_LATENT_ATTENTION", "") not in ("simt", "mma")
 # A step whose portions bring fewer (token, head) rows than this runs them through the mma.sync kernel (blocks of 32 rows)
-LATENT_TC_MIN_ROWS = 2048
+LATENT_TC_MIN_ROWS = 256
 
 
 def latent_tensor_cores(dtype: torch.dtype, d: int, dv: Optional[int], nkv: int = 1, softcap: Optional[float] = None) -> bool:
@@ -591,7 +594,7 @@ def latent_tensor_cores(dtype: torch.dtype, d: int, dv: Optional[int], nkv: int 
 
 
 def latent_tcgen05(dtype: torch.dtype, d: int, dv: Optional[int], page_size: int, nkv: int = 1, softcap: Optional[float] = None) -> bool:
-    """Whether the tcgen05 kernel for prompt portions over cached latents takes these sizes (rows and values of whole 16-byte
+    """Whether the tcgen05 kernel for attention over cached latents takes these sizes (rows and values of whole 16-byte
     pieces, rows of up to 640 numbers, pages of a multiple of 64 positions)."""
     return (_TC_LATENT and latent_tensor_cores(dtype, d, dv, nkv, softcap)
             and bool(library().lily_latent_attention_tc_takes(int(d), int(dv), int(page_size))))
@@ -798,7 +801,13 @@ def attention_decode(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch
     common = (_p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"), block_table.shape[-1],
               _i32(seq_lens, "seq_lens"), _p(scratch), requests, splits, nq, nkv, d, page_size, int(window or 0),
               float(scale))
-    if values_in_keys and latent_tensor_cores(q.dtype, d, dv, nkv, softcap) and not stages:
+    if values_in_keys and latent_tcgen05(q.dtype, d, dv, page_size, nkv, softcap) and not stages:
+        _call("lily_latent_attention_decode_tc", _p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"),
+              block_table.shape[-1], _i32(seq_lens, "seq_lens"), _p(scratch), requests, splits, nq, d, dv, page_size,
+              int(window or 0), float(scale), kv_layer.shape[0], _stream())
+        if splits > 1:
+            _call("lily_attention_combine", _p(scratch), _p(out), requests, nq, dv, splits, _dt(q), _stream())
+    elif values_in_keys and latent_tensor_cores(q.dtype, d, dv, nkv, softcap) and not stages:
         _call("lily_latent_attention_decode_mma", _p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"),
               block_table.shape[-1], _i32(seq_lens, "seq_lens"), _p(scratch), requests, splits, nq, d, dv, page_size,
               int(window or 0), float(scale), _stream())
@@ -874,6 +883,17 @@ def choose_decode_splits(num_decode: int, kv_heads: int, max_seq_len: int, sm_co
     return max(1, min(limit, -(-4 * held // pairs)))
 
 
+def choose_latent_splits(requests: int, heads: int, rank: int, max_seq_len: int, sm_count: int = 148) -> int:
+    """Key ranges of a decode row over cached latents on the tcgen05 kernel, which has one block a SM and walks tiles of 128
+    keys: the count that ends first, a block costing its tiles and about two more
+    (queries, first tile, results) and a range its share of the merge (measured: one row of 4,096 keys of 576 numbers,
+    32 heads: 16 ranges 20.9 us, 32 ranges 27.0, 8 ranges 22.3)."""
+    units = requests * -(-heads // 128) * (-(-rank // 256))
+    tiles = max(1, -(-max_seq_len // 128))
+    cost = lambda s: -(-units * s // sm_count) * (-(-tiles // s) + 2) + 0.07 * s
+    return min(range(1, min(tiles, 64) + 1), key=cost)
+
+
 @dataclass(frozen=True)
 class DecodePlan:
     """How the decode attention of a step runs (the same for every layer of a cache group)."""
@@ -905,7 +925,7 @@ def whole_rows_pay(pairs: int, sm_count: int = 148) -> bool:
 
 def plan_decode_attention(dtype: torch.dtype, requests: int, nq: int, nkv: int, d: int, max_seq_len: int,
                           even: bool = False, dv: Optional[int] = None, values_in_keys: bool = False,
-                          keep_first: int = 0, fusable: bool = True, cuda_cores: bool = False) -> DecodePlan:
+                          keep_first: int = 0, fusable: bool = True, cuda_cores: bool = False, page_size: int = 0) -> DecodePlan:
     """The plan for ``requests`` rows that bring one token each, none longer than ``max_seq_len`` positions.
     A step in which every request brings one token may hand the qkv product straight to the attention kernel
     (``fused``): every block then finishes its own queries, which costs less than a kernel of its own while all
@@ -913,6 +933,7 @@ def plan_decode_attention(dtype: torch.dtype, requests: int, nq: int, nkv: int, 
     2 % of the step).
     ``cuda_cores``: the attention has options only the CUDA-core kernel has (a sink, values of all kv heads; ``dv`` is
     then the width of a head's output row).
+    ``page_size``: of a cache of latents (``values_in_keys``), which says whether the tcgen05 kernel takes it.
     ``fusable`` False: the caller prepares queries and cache itself (something stands between its projection and
     the attention); ``keep_first``: the window keeps the first positions in sight (the caller then prepares queries
     and cache itself as well).
@@ -924,6 +945,9 @@ def plan_decode_attention(dtype: torch.dtype, requests: int, nq: int, nkv: int, 
         return DecodePlan(1, False, 0, "single")
     group = nq // nkv
     dv = int(dv or d)
+    if values_in_keys and page_size and latent_tcgen05(dtype, d, dv, page_size, nkv):
+        splits = choose_latent_splits(requests, nq, dv, max_seq_len, sm_count())
+        return DecodePlan(splits, False, decode_scratch_floats(requests, nq, dv, splits), "single" if splits == 1 else "wave")
     tensor_cores = dv == d and not values_in_keys and not cuda_cores and uses_tensor_cores(dtype, d)      # values of another head size run on CUDA cores
     fusable = fusable and not keep_first          # the kernel that takes the projection itself has no kept first positions
     row_blocks = -(-group // 16)                 # the tensor-core kernel takes 16 query heads of a kv head a block

@@ -145,7 +145,7 @@ class LatentAttention(Mixer):
         def make(b):
             nd = b.num_decode
             decode = ops.plan_decode_attention(dtype, nd, s.num_heads, 1, s.row, b.max_decode_len, even=b.decode_even,
-                                               dv=s.kv_rank, values_in_keys=True)
+                                               dv=s.kv_rank, values_in_keys=True, page_size=page)
             rows = tiles = None
             if b.num_requests > nd:
                 rows = ops.prefill_tile_rows(dtype, s.row, page, b.num_tokens - nd, dv=s.kv_rank, values_in_keys=True,

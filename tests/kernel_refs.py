@@ -246,7 +246,7 @@ class DecodePlan:
 
 
 def plan_decode_attention(dtype, requests, nq, nkv, d, max_seq_len, even=False, dv=None, values_in_keys=False,
-                          keep_first=0, fusable=True, cuda_cores=False):
+                          keep_first=0, fusable=True, cuda_cores=False, page_size=0):
     if requests == 0:
         return DecodePlan(1, False, 0, "single")
     splits = 2 if max_seq_len >= 32 else 1

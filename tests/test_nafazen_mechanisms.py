@@ -181,6 +181,97 @@ def test_rows_that_stand_out_are_seen():
         assert float((other - want)[20:].abs().max()) > 0.1 * float(want.abs().max())
 
 
+def cached_rows(g, lens, page, row, dtype, scale=0.7):
+    """A cache of random rows for sequences of these lengths, pages handed out in a scrambled order; the rows of each."""
+    pages = [-(-n // page) for n in lens]
+    order = (torch.randperm(sum(pages), generator=g) + 1).tolist()
+    table = torch.zeros(len(lens), max(pages), dtype=torch.int32)
+    at = 0
+    for r, n in enumerate(pages):
+        table[r, :n] = torch.tensor(order[at:at + n], dtype=torch.int32)
+        at += n
+    cache = (torch.randn(sum(pages) + 1, page * row, generator=g) * scale).to(device="cuda", dtype=dtype)
+    rows = cache.float().cpu().view(-1, page, row)
+    return cache, table, [torch.stack([rows[int(table[r, j // page]), j % page] for j in range(n)]) for r, n in enumerate(lens)]
+
+
+def plain_rows_attention(q, keys, first, rank, scale, window):
+    """q [t, heads, row] at positions ``first`` on over keys [n, row]: the values are the first ``rank`` columns."""
+    s = torch.einsum("thd,jd->thj", q, keys) * scale
+    i = torch.arange(first, first + q.shape[0])[:, None, None]
+    j = torch.arange(keys.shape[0])[None, None, :]
+    seen = (j <= i) if window is None else ((j <= i) & (i - j < window))
+    return torch.softmax(s.masked_fill(~seen, float("-inf")), -1) @ keys[:, :rank]
+
+
+TC_SIZES = [(4, 64, 64), (4, 80, 64), (4, 128, 96), (32, 576, 512), (24, 264, 256), (6, 272, 264), (130, 64, 48), (3, 640, 8), (1, 16, 8),
+            (128, 192, 128), (100, 144, 136)]
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("heads,row,rank", TC_SIZES)
+@pytest.mark.parametrize("page,window", [(64, None), (128, 50), (64, 130)])
+def test_portions_over_cached_rows_on_tcgen05(heads, row, rank, page, window):
+    """The tcgen05 kernel against a plain softmax over the rows as they lie in the cache: requests of unequal lengths side
+    by side with and without a cached prefix, tiles that end inside a token group, rows that are no multiple of a piece,
+    ranks in one and two column blocks, more heads than a block has rows; the scores are sharp (a scale of
+    several units), so a wrong key shows."""
+    from lily_b200.csrc import ops
+    dt = torch.bfloat16
+    assert ops.latent_tcgen05(dt, row, rank, page)
+    g = torch.Generator().manual_seed(row)
+    new, prefix = [37, 5, 130 if heads <= 32 else 20], [200, 0, 64]
+    cache, table, keys = cached_rows(g, [a + b for a, b in zip(new, prefix)], page, row, dt)
+    q = torch.randn(sum(new), heads * row, generator=g).to(device="cuda", dtype=dt)
+    out = torch.zeros(sum(new), heads * rank, device="cuda", dtype=dt)
+    scale = 3.0 / math.sqrt(row)
+    tile = int(ops.library().lily_latent_attention_tc_tile_tokens(heads))
+    cu = [0, new[0], new[0] + new[1], sum(new)]
+    tr, ts = ops.prefill_tiles(prefix, new, 0, tile, "cuda")
+    ops.attention_prefill(q, cache, table.cuda(), i32(cu, "cuda"), i32(prefix, "cuda"), tr, ts, out, heads, 1, row, page, scale, window,
+                          tile_rows=tile, dv=rank, values_in_keys=True)
+    for r in range(3):
+        want = plain_rows_attention(q[cu[r]:cu[r + 1]].float().cpu().view(-1, heads, row), keys[r], prefix[r], rank, scale, window)
+        got = out[cu[r]:cu[r + 1]].float().cpu().view(-1, heads, rank)
+        assert float((got - want).abs().max()) < 1e-2 * float(want.abs().max()), r
+    assert ops.latent_attention_status() == 0
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("heads,row,rank", TC_SIZES)
+@pytest.mark.parametrize("window", [None, 140])
+def test_decoding_over_cached_rows_on_tcgen05(heads, row, rank, window):
+    """One new token a request over rows of very different lengths, the keys in one range and in several (some of them
+    without a key for the short requests), and as the plan cuts them."""
+    from lily_b200.csrc import ops
+    dt, page = torch.bfloat16, 64
+    g = torch.Generator().manual_seed(row + 1)
+    lens = [1, 128, 129, 700, 64, 1500]
+    cache, table, keys = cached_rows(g, lens, page, row, dt)
+    q = torch.randn(len(lens), heads * row, generator=g).to(device="cuda", dtype=dt)
+    scale = 3.0 / math.sqrt(row)
+    want = torch.cat([plain_rows_attention(q[r:r + 1].float().cpu().view(1, heads, row), keys[r], n - 1, rank, scale, window)
+                      for r, n in enumerate(lens)])
+    plan = ops.plan_decode_attention(dt, len(lens), heads, 1, row, max(lens), dv=rank, values_in_keys=True, page_size=page)
+    for splits in (1, 2, 5, 12, plan.splits):
+        out = torch.zeros(len(lens), heads * rank, device="cuda", dtype=dt)
+        scratch = torch.empty(max(1, ops.decode_scratch_floats(len(lens), heads, rank, splits)), device="cuda")
+        ops.attention_decode(q, cache, table.cuda(), i32(lens, "cuda"), out, scratch, splits, heads, 1, row, page, scale, window, dv=rank,
+                             values_in_keys=True)
+        got = out.float().cpu().view(len(lens), heads, rank)
+        assert float((got - want).abs().max()) < 1e-2 * float(want.abs().max()), splits
+    assert ops.latent_attention_status() == 0
+
+
+def test_ranges_of_a_decode_step_over_latents():
+    from lily_b200.csrc.ops import choose_latent_splits
+
+    assert choose_latent_splits(8, 32, 512, 4096) == 8 and choose_latent_splits(200, 32, 512, 100) == 1
+    for requests in (1, 3, 40, 500):
+        for length in (1, 128, 1000, 100000):
+            assert 1 <= choose_latent_splits(requests, 16, 256, length) <= max(1, -(-length // 128))
+
+
 @pytest.mark.parametrize("device", DEVICES)
 def test_product_per_head_into_a_view(device):
     ops = ops_for(device)
