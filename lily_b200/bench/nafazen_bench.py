@@ -126,10 +126,10 @@ def kernel_table(z: dict, tokens: int, batch: int, context: int, reps: int = 30,
         del zs, up, down, dense_gu, dense_dn
         # ---- the experts beside the closest model's
         experts, e_ff = 16, z["ff"] // 4
-        router = rnd(experts + 1, width) / width ** 0.5
+        router = (rnd(experts + 8, width) / width ** 0.5).to(dt)
         corr = rnd(experts) / (2 * experts)
         add("moe_route + align (sigmoid, shared gate)", "moe_route + align", [
-            lambda x=x: ops.moe_route(x, router, None, 3, experts, scores="sigmoid", renormalise=False, shared_gate=True) for x in xs],
+            lambda x=x: ops.moe_route(x, router, None, 3, experts, scores="sigmoid", renormalise=False, shared_gate=True, outputs=experts) for x in xs],
             n * width * 2 + (experts + 1) * width * 4, 2.0 * n * (experts + 1) * width, fp32_tflops, shape=label)
         router_g = router[:experts].contiguous()
         add("moe_route + align (Godotar)", "-", [lambda x=x: ops.moe_route(x, router_g, corr, 4, experts) for x in xs],
@@ -137,7 +137,7 @@ def kernel_table(z: dict, tokens: int, batch: int, context: int, reps: int = 30,
         gu, dn = (rnd(experts, 2 * e_ff, width) / width ** 0.5).to(dt), (rnd(experts, width, e_ff) / e_ff ** 0.5).to(dt)
         for name, like, top in (("moe_experts (weights on inputs, shared)", "moe_experts", 3), ("moe_experts (Godotar)", "-", 4)):
             ours = top == 3
-            routed = [ops.moe_route(x, router, None, top, experts, scores="sigmoid", renormalise=False, shared_gate=True) if ours
+            routed = [ops.moe_route(x, router, None, top, experts, scores="sigmoid", renormalise=False, shared_gate=True, outputs=experts) if ours
                       else ops.moe_route(x, router_g, corr, top, experts) for x in xs]
             how = dict(activation="silu", weight_on_input=True, shared=xs[0]) if ours else dict(limit=7.0, alpha=1.702)
             pairs = n * top

@@ -25,6 +25,80 @@ namespace lily {
 constexpr int ROUTE_MAX = 1024;       // router outputs
 constexpr int ROUTE_TOP_MAX = 64;
 
+// Scores and choice of token t by one warp.  s: the token's logits in shared memory (overwritten), `outputs` of them and, with
+// `gate`, the shared gate's behind them; picked: room for `top` numbers.
+__device__ __forceinline__ void choose_experts(float* s, int t, int outputs, const float* __restrict__ correction, int top, int sigmoid,
+                                               int renormalise, float* picked, int* __restrict__ chosen, float* __restrict__ weights,
+                                               float* __restrict__ gate) {
+    const int lane = threadIdx.x & 31, rows = outputs + (gate ? 1 : 0);
+    float inv = 1.f;
+    if (sigmoid) {
+        for (int e = lane; e < rows; e += 32) {
+            const float p = 1.f / (1.f + expf(-s[e]));
+            s[e] = p;
+            if (e == outputs) gate[t] = p;
+        }
+    } else {
+        float mx = -INFINITY;
+        for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, s[e]);
+        mx = warp_max(mx);
+        float sum = 0.f;
+        for (int e = lane; e < outputs; e += 32) {
+            const float p = expf(s[e] - mx);
+            s[e] = p;
+            sum += p;
+        }
+        sum = warp_sum(sum);
+        inv = 1.f / sum;
+        if (gate && lane == 0) gate[t] = 1.f / (1.f + expf(-s[outputs]));
+    }
+    __syncwarp();
+    float total = 0.f;
+    for (int k = 0; k < top; ++k) {
+        float best = -INFINITY;
+        int at = outputs;
+        for (int e = lane; e < outputs; e += 32) {
+            const float p = s[e];
+            if (p < 0.f) continue;                                // taken already
+            const float c = correction ? p * inv + correction[e] : p * inv;
+            if (c > best) { best = c; at = e; }
+        }
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+            if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+        }
+        if (at >= outputs) at = 0;                                // cannot happen while top <= outputs
+        const float p = s[at] * inv;
+        total += p;
+        __syncwarp();
+        if (lane == 0) {
+            chosen[(size_t)t * top + k] = at;
+            picked[k] = p;
+            s[at] = -1.f;
+        }
+        __syncwarp();
+    }
+    const float norm = renormalise ? 1.f / (total + 1e-20f) : 1.f;
+    for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] = picked[k] * norm;
+    __syncwarp();
+}
+
+// The choice from logits that a product has left (finished rows or partial sums).  grid (ceil(tokens / 4)), block 128: a
+// warp a token.
+__global__ void moe_choose_kernel(const Operand logits, int ld, int tokens, const float* __restrict__ correction, int outputs, int top, int sigmoid,
+                                  int renormalise, int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ gate) {
+    __shared__ float picked[4][ROUTE_TOP_MAX];
+    extern __shared__ __align__(16) float dyn[];             // [4][rows]
+    pdl_enter_small();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 4 + warp, rows = outputs + (gate ? 1 : 0);
+    if (t >= tokens) return;
+    float* s = dyn + warp * rows;
+    for (int e = lane; e < rows; e += 32) s[e] = logits((size_t)t * ld + e);
+    __syncwarp();
+    choose_experts(s, t, outputs, correction, top, sigmoid, renormalise, picked[warp], chosen, weights, gate);
+}
+
 // grid (ceil(tokens / TB)), block 128: a block takes TB tokens, so a number of the router matrix read once serves TB
 // sums (one token a block rereads the matrix from L2 for every token: 50 us for 2,048 tokens of 2,048 columns).
 // A token's logits are summed in the same order whatever TB is.
@@ -106,62 +180,8 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int tokens, int width,
         }
     }
     __syncthreads();
-    // scores and choice: a warp a token
-    for (int j = warp; j < nt; j += nwarp) {
-        float* s = sc + j * rows;
-        const int t = t0 + j;
-        float inv = 1.f;
-        if (sigmoid) {
-            for (int e = lane; e < rows; e += 32) {
-                const float p = 1.f / (1.f + expf(-s[e]));
-                s[e] = p;
-                if (e == outputs) gate[t] = p;
-            }
-        } else {
-            float mx = -INFINITY;
-            for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, s[e]);
-            mx = warp_max(mx);
-            float sum = 0.f;
-            for (int e = lane; e < outputs; e += 32) {
-                const float p = expf(s[e] - mx);
-                s[e] = p;
-                sum += p;
-            }
-            sum = warp_sum(sum);
-            inv = 1.f / sum;
-            if (gate && lane == 0) gate[t] = 1.f / (1.f + expf(-s[outputs]));
-        }
-        __syncwarp();
-        float total = 0.f;
-        for (int k = 0; k < top; ++k) {
-            float best = -INFINITY;
-            int at = outputs;
-            for (int e = lane; e < outputs; e += 32) {
-                const float p = s[e];
-                if (p < 0.f) continue;                                // taken already
-                const float c = correction ? p * inv + correction[e] : p * inv;
-                if (c > best) { best = c; at = e; }
-            }
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-                if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
-            }
-            if (at >= outputs) at = 0;                                // cannot happen while top <= outputs
-            const float p = s[at] * inv;
-            total += p;
-            __syncwarp();
-            if (lane == 0) {
-                chosen[(size_t)t * top + k] = at;
-                picked[warp][k] = p;
-                s[at] = -1.f;
-            }
-            __syncwarp();
-        }
-        const float norm = renormalise ? 1.f / (total + 1e-20f) : 1.f;
-        for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] = picked[warp][k] * norm;
-        __syncwarp();
-    }
+    for (int j = warp; j < nt; j += nwarp)
+        choose_experts(sc + j * rows, t0 + j, outputs, correction, top, sigmoid, renormalise, picked[warp], chosen, weights, gate);
 }
 
 // One block of 1024 threads.  chosen [pairs]; experts: router outputs that have weights (the rest are skipped here).
@@ -411,6 +431,20 @@ LILY_API int lily_moe_route(const void* h, int tokens, int width, const float* r
     else { if (tb == 4) GO(float, 4); else GO(float, 1); }
 #undef GO
     LILY_CHECK_LAUNCH("moe_route");
+    return 0;
+}
+
+// The same from the logits: rows `ld` apart, outputs (+ 1 with `gate`) of them read.
+LILY_API int lily_moe_choose(const void* logits, int logits_dtype, int splits, size_t stride, int ld, int tokens, const float* correction, int outputs,
+                             int top, int sigmoid, int renormalise, int* chosen, float* weights, float* gate, cudaStream_t stream) {
+    if (tokens == 0) return 0;
+    LILY_REQUIRE(outputs >= 1 && outputs <= ROUTE_MAX, "moe_choose: %d router outputs (up to %d)", outputs, ROUTE_MAX);
+    LILY_REQUIRE(top >= 1 && top <= outputs && top <= ROUTE_TOP_MAX, "moe_choose: top %d of %d", top, outputs);
+    LILY_REQUIRE(splits >= 1 && logits_dtype == kF32 && ld >= outputs + (gate ? 1 : 0), "moe_choose: float32 logits in rows of %d", ld);
+    const Operand x{logits, 0, splits, stride};
+    launch_pdl(moe_choose_kernel, dim3((tokens + 3) / 4), dim3(128), (size_t)4 * (outputs + 1) * sizeof(float), stream, x, ld, tokens, correction,
+               outputs, top, sigmoid, renormalise, chosen, weights, gate);
+    LILY_CHECK_LAUNCH("moe_choose");
     return 0;
 }
 

@@ -75,6 +75,7 @@ _SIGNATURES = {
     "lily_latent_query": [_vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _vp],
     "lily_head_gate": [_vp, _i, _vp, _i, _i, _sz, _i, _i, _i, _i, _i, _vp, _i, _vp],
     "lily_moe_route": [_vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp],
+    "lily_moe_choose": [_vp, _i, _i, _sz, _i, _i, _vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp],
     "lily_moe_align": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp],
     "lily_moe_gemm": [_i, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _i, _f, _f, _vp, _i, _vp],
     "lily_moe_combine": [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _sz, _vp, _vp, _i, _vp],
@@ -1486,18 +1487,24 @@ class ExpertRouting:
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, experts: int,
-              scores: str = "softmax", renormalise: bool = True, shared_gate: bool = False) -> ExpertRouting:
-    """Scores of all router outputs (float32 logits ``router . h``; their softmax, or with ``scores`` "sigmoid" each one's
+              scores: str = "softmax", renormalise: bool = True, shared_gate: bool = False,
+              outputs: Optional[int] = None) -> ExpertRouting:
+    """Scores of all router outputs (float32 logits ``router . h``, by this package's kernel for a float32 matrix; a matrix in
+    ``h``'s bfloat16 takes a product with a float32 result, whose terms are exact; their softmax, or with ``scores`` "sigmoid" each one's
     sigmoid), the ``top`` largest scores (+ correction) chosen, their weights the scores themselves, over their sum with
     ``renormalise``; then the pairs of the first ``experts`` outputs (those with weights; the rest stand for the identity)
     grouped by expert.  ``shared_gate``: the matrix has one more row, the sigmoid of whose product is the token's gate for
-    the shared expert."""
+    the shared expert.  ``outputs``: how many the router has where the matrix goes on behind its own rows (a bfloat16 matrix
+    whose rows are padded to a multiple of 8 gets the library's faster product)."""
     _dev(h, router, correction)
     tokens, width = h.shape
-    outputs = router.shape[0] - (1 if shared_gate else 0)
-    if (router.dtype != torch.float32 or router.shape[1] != width
+    if outputs is None:
+        outputs = router.shape[0] - (1 if shared_gate else 0)
+    if router.shape[0] < outputs + (1 if shared_gate else 0):
+        raise KernelError(f"moe_route: a matrix of {router.shape[0]} rows for {outputs} outputs")
+    if (router.dtype not in (torch.float32, h.dtype) or router.shape[1] != width
             or (correction is not None and (correction.dtype != torch.float32 or correction.numel() != outputs))):
-        raise KernelError("moe_route: router [outputs, width] and correction [outputs] are float32")
+        raise KernelError("moe_route: router [outputs, width] in float32 or the input's dtype, correction [outputs] float32")
     if scores not in ("softmax", "sigmoid"):
         raise KernelError(f"moe_route: no scores {scores!r} (have softmax, sigmoid)")
     dev = h.device
@@ -1509,8 +1516,14 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.
         ints, [pairs, pairs, pairs, experts + 1, max_tiles, max_tiles, 1])
     weights = torch.empty((tokens, top), dtype=torch.float32, device=dev)
     gate = torch.empty((tokens,), dtype=torch.float32, device=dev) if shared_gate else None
-    _call("lily_moe_route", _p(h), tokens, width, _p(router), _p(correction), outputs, top, int(scores == "sigmoid"), int(renormalise),
-          _p(chosen), _p(weights), _p(gate), _dt(h), _stream())
+    how = (outputs, top, int(scores == "sigmoid"), int(renormalise), _p(chosen), _p(weights), _p(gate))
+    if router.dtype == torch.bfloat16:
+        z = linear_split(h, router)
+        if z is None:
+            z = linear(h, router, out_dtype=torch.float32)
+        _call("lily_moe_choose", *_operand(z, tokens, router.shape[0], "moe_route"), router.shape[0], tokens, _p(correction), *how, _stream())
+    else:
+        _call("lily_moe_route", _p(h), tokens, width, _p(router), _p(correction), *how, _dt(h), _stream())
     _call("lily_moe_align", _p(chosen), pairs, experts, _p(offsets), _p(order), _p(place), _p(tile_expert), _p(tile_row),
           _p(tile_count), max_tiles, _stream())
     return ExpertRouting(chosen.view(tokens, top), weights, offsets, order, place, tile_expert, tile_row, tile_count,

@@ -97,12 +97,15 @@ class RoutedExperts(FeedForward):
 
     def load(self, get) -> None:
         s, p = self.spec, self.prefix
-        self.router = get(f"{p}.{s.name('router')}").float().contiguous()           # the router works in float32
+        # the logits are float32 sums of exact terms either way (a router matrix is served in the compute dtype)
+        self.router = get(f"{p}.{s.name('router')}").contiguous()
         if s.correction:
             self.correction = get(f"{p}.{s.name('correction')}").float().contiguous()
         if self.shared is not None:
             self.shared.load(get)
-            self.router = torch.cat([self.router, get(f"{p}.{s.name('shared_gate')}").float()], 0).contiguous()
+            self.router = torch.cat([self.router, get(f"{p}.{s.name('shared_gate')}")], 0).contiguous()
+        if self.router.dtype == torch.bfloat16 and self.router.shape[0] % 8:
+            self.router = torch.cat([self.router, self.router.new_zeros(-self.router.shape[0] % 8, s.hidden_size)], 0).contiguous()
         ff, h = s.intermediate_size, s.hidden_size
         if s.experts:
             first = get(self._expert(0, "gate"))
@@ -118,7 +121,7 @@ class RoutedExperts(FeedForward):
     def forward(self, x, batch):
         s, ops = self.spec, self.ctx.ops
         routing = ops.moe_route(x, self.router, self.correction, s.top, s.experts, scores=s.scores, renormalise=s.renormalise,
-                                shared_gate=self.shared is not None)
+                                shared_gate=self.shared is not None, outputs=s.outputs)
         shared = None if self.shared is None else self.shared.forward(x, batch)
         out = ops.moe_experts(x, routing, self.w_gate_up, self.w_down, s.limit, s.alpha, activation=s.activation,
                               weight_on_input=s.weight_on == "input", shared=shared)

@@ -583,11 +583,11 @@ class ExpertRouting:
     gate: Optional[torch.Tensor] = None
 
 
-def moe_route(h, router, correction, top, experts, scores="softmax", renormalise=True, shared_gate=False):
+def moe_route(h, router, correction, top, experts, scores="softmax", renormalise=True, shared_gate=False, outputs=None):
     z = h.float() @ router.float().t()
-    gate = None
-    if shared_gate:
-        z, gate = z[:, :-1], torch.sigmoid(z[:, -1])
+    outputs = router.shape[0] - int(shared_gate) if outputs is None else outputs
+    gate = torch.sigmoid(z[:, outputs]) if shared_gate else None
+    z = z[:, :outputs]
     s = torch.softmax(z, -1) if scores == "softmax" else torch.sigmoid(z)
     chosen = torch.topk(s if correction is None else s + correction.float(), top, dim=-1).indices
     picked = torch.gather(s, 1, chosen)

@@ -409,7 +409,7 @@ def test_routed_experts_with_weights_on_their_inputs(device, experts, top, ff, w
         ops = ops_for(device)
         big = n(1100, width)                                                  # several tokens share a block on the GPU
         routing = ops.moe_route(big.to(device=device, dtype=dtype), part.router, None, top, experts, scores="sigmoid", renormalise=False,
-                                shared_gate=bool(shared))
+                                shared_gate=bool(shared), outputs=experts)
         chosen, weights = pn.route(rounded(big, dtype), wr, "p", top)
         assert torch.equal(routing.chosen.cpu().long().sort(-1).values, chosen.sort(-1).values)
         order = routing.chosen.cpu().long().argsort(-1)
