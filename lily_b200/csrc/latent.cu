@@ -21,7 +21,15 @@ namespace lily {
 // partial sums of a split-k product): the query latent at column q0 (q_rank columns), the key/value latent at kv0
 // (rank columns) followed by the part to rotate (rot columns, of which the first rd are rotated in halves and the
 // rest pass).  The row is read once: what the norms need again stands in shared memory.
-template <typename T>
+template <typename T> __device__ __forceinline__ void put_four(T* dst, float a, float b, float c, float d);
+template <> __device__ __forceinline__ void put_four<float>(float* dst, float a, float b, float c, float d) { *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d); }
+template <> __device__ __forceinline__ void put_four<__nv_bfloat16>(__nv_bfloat16* dst, float a, float b, float c, float d) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+    *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+
+// VEC 4: columns, sizes and rows of whole pieces of four numbers, bases aligned to them.
+template <typename T, int VEC>
 __global__ void latent_prepare_kernel(const Operand in, int ld, int q0, int q_rank, int kv0, int rank, int rot,
                                       int rd, const float* __restrict__ q_gain, const float* __restrict__ kv_gain,
                                       float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
@@ -35,12 +43,26 @@ __global__ void latent_prepare_kernel(const Operand in, int ld, int q0, int q_ra
     const size_t row = (size_t)t * ld;
     float* kv = held + q_rank;
     float ssq = 0.f, ssk = 0.f;
-    for (int c = threadIdx.x; c < q_rank; c += blockDim.x) {
-        const float x = in(row + q0 + c);
-        held[c] = x;
-        ssq = fmaf(x, x, ssq);
+    if (VEC == 4) {
+        for (int c = threadIdx.x * 4; c < q_rank; c += blockDim.x * 4) {
+            const float4 x = in.four(row + q0 + c);
+            *reinterpret_cast<float4*>(held + c) = x;
+            ssq += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+        }
+        if (write_kv)
+            for (int c = threadIdx.x * 4; c < rank + rot; c += blockDim.x * 4) {
+                const float4 x = in.four(row + kv0 + c);
+                *reinterpret_cast<float4*>(kv + c) = x;
+                if (c < rank) ssk += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+            }
+    } else {
+        for (int c = threadIdx.x; c < q_rank; c += blockDim.x) {
+            const float x = in(row + q0 + c);
+            held[c] = x;
+            ssq = fmaf(x, x, ssq);
+        }
     }
-    if (write_kv)
+    if (VEC == 1 && write_kv)
         for (int c = threadIdx.x; c < rank + rot; c += blockDim.x) {
             const float x = in(row + kv0 + c);
             kv[c] = x;
@@ -59,15 +81,27 @@ __global__ void latent_prepare_kernel(const Operand in, int ld, int q0, int q_ra
         ssk += sums[1][w];
     }
     const float inv_q = rsqrtf(ssq / (float)q_rank + eps);
-    for (int c = threadIdx.x; c < q_rank; c += blockDim.x) cq[(size_t)t * q_rank + c] = from_float<T>((held[c] * inv_q) * q_gain[c]);
+    if (VEC == 4)
+        for (int c = threadIdx.x * 4; c < q_rank; c += blockDim.x * 4) {
+            const float4 x = *reinterpret_cast<const float4*>(held + c), g = *reinterpret_cast<const float4*>(q_gain + c);
+            put_four<T>(cq + (size_t)t * q_rank + c, x.x * inv_q * g.x, x.y * inv_q * g.y, x.z * inv_q * g.z, x.w * inv_q * g.w);
+        }
+    else
+        for (int c = threadIdx.x; c < q_rank; c += blockDim.x) cq[(size_t)t * q_rank + c] = from_float<T>((held[c] * inv_q) * q_gain[c]);
     if (!write_kv) return;
     const float inv_kv = rsqrtf(ssk / (float)rank + eps);
     const int pos = positions[t];
     const int page = block_table[(size_t)token_req[t] * bt_stride + pos / page_size];
     const int width = rank + rot;
     T* dst = layer + ((size_t)page * page_size + pos % page_size) * width;
-    for (int c = threadIdx.x; c < rank; c += blockDim.x)
-        dst[c] = from_float<T>((kv[c] * inv_kv) * kv_gain[c]);
+    if (VEC == 4)
+        for (int c = threadIdx.x * 4; c < rank; c += blockDim.x * 4) {
+            const float4 x = *reinterpret_cast<const float4*>(kv + c), g = *reinterpret_cast<const float4*>(kv_gain + c);
+            put_four<T>(dst + c, x.x * inv_kv * g.x, x.y * inv_kv * g.y, x.z * inv_kv * g.z, x.w * inv_kv * g.w);
+        }
+    else
+        for (int c = threadIdx.x; c < rank; c += blockDim.x)
+            dst[c] = from_float<T>((kv[c] * inv_kv) * kv_gain[c]);
     const int half = rd / 2;
     const float* kr = kv + rank;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
@@ -82,7 +116,8 @@ __global__ void latent_prepare_kernel(const Operand in, int ld, int q0, int q_ra
 // One block per token.  q [tokens, heads, d + rot]: the up-projected queries, of which the last rot columns of a head are
 // rotated into the last rot columns of the head's row of out [tokens, heads, rank + rot] (the first rank are the
 // unrotated part carried into the latent's space, which the per-head product has written).
-template <typename T>
+// VEC 2 (bfloat16): two neighbouring pairs a thread.
+template <typename T, int VEC>
 __global__ void latent_query_kernel(const T* __restrict__ q, int heads, int d, int rank, int rot, int rd,
                                     const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                                     const int* __restrict__ positions, T* __restrict__ out) {
@@ -90,7 +125,20 @@ __global__ void latent_query_kernel(const T* __restrict__ q, int heads, int d, i
     const int t = blockIdx.x, pos = positions[t], half = rd / 2, rest = rot - rd;
     const T* src = q + (size_t)t * heads * (d + rot) + d;
     T* dst = out + (size_t)t * heads * (rank + rot) + rank;
-    for (int n = threadIdx.x; n < heads * half; n += blockDim.x) {
+    if (VEC == 2) {
+        const int pairs = half / 2;
+        for (int n = threadIdx.x; n < heads * pairs; n += blockDim.x) {
+            const int h = n / pairs, i = n % pairs * 2;
+            const __nv_bfloat16* qr = reinterpret_cast<const __nv_bfloat16*>(src) + (size_t)h * (d + rot) + i;
+            __nv_bfloat16* to = reinterpret_cast<__nv_bfloat16*>(dst) + (size_t)h * (rank + rot) + i;
+            const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(qr));
+            const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(qr + half));
+            const float2 c = *reinterpret_cast<const float2*>(cos_t + (size_t)pos * half + i);
+            const float2 s = *reinterpret_cast<const float2*>(sin_t + (size_t)pos * half + i);
+            *reinterpret_cast<__nv_bfloat162*>(to) = __floats2bfloat162_rn(u.x * c.x - v.x * s.x, u.y * c.y - v.y * s.y);
+            *reinterpret_cast<__nv_bfloat162*>(to + half) = __floats2bfloat162_rn(v.x * c.x + u.x * s.x, v.y * c.y + u.y * s.y);
+        }
+    } else for (int n = threadIdx.x; n < heads * half; n += blockDim.x) {
         const int h = n / half, i = n % half;
         const T* qr = src + (size_t)h * (d + rot);
         T* to = dst + (size_t)h * (rank + rot);
@@ -137,13 +185,14 @@ LILY_API int lily_latent_prepare(const void* in, int in_dtype, int in_splits, si
     LILY_REQUIRE(smem <= 47 * 1024, "latent_prepare: latents of %d and %d columns do not fit a block's shared memory", q_rank, rank + rot);
     const int widest = q_rank > rank + rot ? q_rank : rank + rot;
     dim3 grid(tokens), block(tokens <= 64 && widest > 512 ? 512 : 128);
-    if (dtype == kBF16)
-        launch_pdl(latent_prepare_kernel<__nv_bfloat16>, grid, block, smem, stream, x, ld, q0, q_rank, kv0, rank, rot, rd, q_gain, kv_gain,
-                   eps, cos_t, sin_t, positions, token_req, block_table, bt_stride, (__nv_bfloat16*)layer, page_size, write_kv,
-                   (__nv_bfloat16*)cq);
-    else
-        launch_pdl(latent_prepare_kernel<float>, grid, block, smem, stream, x, ld, q0, q_rank, kv0, rank, rot, rd, q_gain, kv_gain, eps,
-                   cos_t, sin_t, positions, token_req, block_table, bt_stride, (float*)layer, page_size, write_kv, (float*)cq);
+    const bool vec = q_rank % 4 == 0 && rank % 4 == 0 && rot % 4 == 0 && q0 % 4 == 0 && kv0 % 4 == 0 && ld % 4 == 0 && x.vector_ok() &&
+                     ((uintptr_t)cq & 15) == 0 && ((uintptr_t)layer & 15) == 0 && ((uintptr_t)q_gain & 15) == 0 && ((uintptr_t)kv_gain & 15) == 0;
+#define GO(T, V)                                                                                                                \
+    launch_pdl(latent_prepare_kernel<T, V>, grid, block, smem, stream, x, ld, q0, q_rank, kv0, rank, rot, rd, q_gain, kv_gain, eps, \
+               cos_t, sin_t, positions, token_req, block_table, bt_stride, (T*)layer, page_size, write_kv, (T*)cq)
+    if (dtype == kBF16) { if (vec) GO(__nv_bfloat16, 4); else GO(__nv_bfloat16, 1); }
+    else { if (vec) GO(float, 4); else GO(float, 1); }
+#undef GO
     LILY_CHECK_LAUNCH("latent_prepare");
     return 0;
 }
@@ -155,11 +204,16 @@ LILY_API int lily_latent_query(const void* q, int tokens, int heads, int d, int 
     LILY_REQUIRE(rd == 0 || (cos_t && sin_t), "latent_query: rotation needs its tables");
     const int work = heads * (rd / 2 > rot - rd ? rd / 2 : rot - rd);
     dim3 grid(tokens), block(work >= 512 ? 512 : (work >= 128 ? 128 : 32));
-    if (dtype == kBF16)
-        launch_pdl(latent_query_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)q, heads, d, rank, rot, rd, cos_t,
+    const bool two = dtype == kBF16 && rd % 4 == 0 && rd > 0 && d % 2 == 0 && rot % 2 == 0 && rank % 2 == 0 && ((uintptr_t)q & 3) == 0 &&
+                     ((uintptr_t)out & 3) == 0 && ((uintptr_t)cos_t & 7) == 0 && ((uintptr_t)sin_t & 7) == 0;
+    if (two)
+        launch_pdl(latent_query_kernel<__nv_bfloat16, 2>, grid, block, 0, stream, (const __nv_bfloat16*)q, heads, d, rank, rot, rd, cos_t,
+                   sin_t, positions, (__nv_bfloat16*)out);
+    else if (dtype == kBF16)
+        launch_pdl(latent_query_kernel<__nv_bfloat16, 1>, grid, block, 0, stream, (const __nv_bfloat16*)q, heads, d, rank, rot, rd, cos_t,
                    sin_t, positions, (__nv_bfloat16*)out);
     else
-        launch_pdl(latent_query_kernel<float>, grid, block, 0, stream, (const float*)q, heads, d, rank, rot, rd, cos_t, sin_t, positions,
+        launch_pdl(latent_query_kernel<float, 1>, grid, block, 0, stream, (const float*)q, heads, d, rank, rot, rd, cos_t, sin_t, positions,
                    (float*)out);
     LILY_CHECK_LAUNCH("latent_query");
     return 0;
