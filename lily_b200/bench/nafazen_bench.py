@@ -40,7 +40,7 @@ def nafazen_config(z: dict, layers: int) -> dict:
     kinds = [{"type": "latent_attention", "mixer": scaled, "mlp": dense}, {"type": "latent_attention_2", "mixer": own, "mlp": moe},
              {"type": "latent_attention", "mixer": scaled, "mlp": dense}, {"type": "latent_attention_2", "mixer": reader, "mlp": moe}]
     return {"architecture": "Nafazen", "vocab": z["vocab"], "width": z["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
-            "logit_softcap": 30.0, "layers": [kinds[i % 4] for i in range(layers)]}
+            "logit_softcap": 25.0, "layers": [kinds[i % 4] for i in range(layers)]}
 
 
 def closest_config(z: dict, layers: int) -> dict:

@@ -50,7 +50,7 @@ VARIED = {"architecture": "Nafazen", "vocab": 131, "width": 48, "norm": {"eps": 
 # Sharp attention: a large scale puts nearly all weight on the best visible key, so a key that is lost, rotated by another
 # angle or read from another layer's rows changes the output outright.
 SHARP = {"architecture": "Nafazen", "vocab": 97, "width": 32, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
-         "logit_softcap": 30.0,
+         "logit_softcap": 20.0,
          "layers": [layer("latent_attention_2", heads=2, dim=8, rot_dim=8, vdim=8, q_rank=16, kv_rank=16, scale=3.0, mlp=dense(32)),
                     layer("latent_attention_2", heads=3, dim=4, rot_dim=8, vdim=4, q_rank=12, kv_rank=16, scale=3.0, kv_from=0, mlp=dense(24)),
                     layer(heads=1, dim=16, rot_dim=2, vdim=16, q_rank=8, kv_rank=32, scale=3.0, yarn=YARN, mlp=dense(32))]}
@@ -93,7 +93,7 @@ def random_config(seed: int) -> dict:
     cfg = {"architecture": "Nafazen", "vocab": rng.choice([61, 128, 300]), "width": width, "norm": {"eps": rng.choice([1e-5, 1e-6])},
            "embedding": {"scale": rng.choice([0.25, 1.0, 3.0])}, "layers": layers}
     if rng.random() < 0.7:
-        cfg["logit_softcap"] = rng.choice([5.0, 30.0])
+        cfg["logit_softcap"] = rng.choice([5.0, 25.0])
     return cfg
 
 
