@@ -25,6 +25,7 @@ struct AttnArgs {
     const void* qkv;          // [planes][requests, (nq + 2 nkv) d]: float32 partial sums, or bfloat16 with one plane
     int qkv_planes, qkv_f32;
     size_t qkv_stride;        // elements between planes
+    int qkv_ld;               // elements between rows (0: the row is the heads alone)
     const void* q_gain;       // [d] per-head RMSNorm gains (both or none), float32 or bfloat16
     const void* k_gain;
     int gain_f32;
@@ -44,6 +45,7 @@ struct AttnArgs {
                               // with the value heads shifted by x / decode_rows and writes row x of `out` and of the scratch
                               // (planes of decode_rows rows: a step in which every request brings one token)
     int sink;                 // CUDA-core and mma.sync kernels: the softmax's denominator holds one more unit (a key of score 0 without a value)
+    const float* sinks;       // [nq], CUDA-core kernels: the same unit's logarithm, one learned number a query head (null: 0)
     int v_all;                // CUDA-core kernels: a query head is weighted over the values of every kv head, not only its own:
                               // its output row is [nkv][dv] (the caller mixes heads afterwards); `dv` stays one head's size
     int out_f32;              // CUDA-core kernels: outputs are written in float32 whatever the cache's dtype

@@ -235,7 +235,7 @@ attention_mma_kernel(const AttnArgs a, const int page_shift) {
         // range holds this step's position also finishes the key and the value and writes them to their page
         for (int i = tid; i < (BM - nrows) * CH; i += THREADS)
             *reinterpret_cast<uint4*>(q_s + swz<D>(nrows + i / CH, i % CH)) = make_uint4(0, 0, 0, 0);
-        const size_t width = (size_t)(a.nq + 2 * a.nkv) * D;
+        const size_t width = a.qkv_ld ? (size_t)a.qkv_ld : (size_t)(a.nq + 2 * a.nkv) * D;
         auto in = [&](size_t idx) -> float {
             if (!a.qkv_f32) return __bfloat162float(((const __nv_bfloat16*)a.qkv)[idx]);
             const float* p = (const float*)a.qkv + idx;
@@ -927,7 +927,9 @@ LILY_API int lily_attention_decode_mma_fused(const void* qkv, int qkv_planes, si
                                              void* kv, void* out, const int* block_table, int bt_stride,
                                              const int* seq_lens, float* scratch, int requests, int splits, int nq,
                                              int nkv, int d, int page_size, int window, float scale, int stages,
-                                             float softcap, cudaStream_t stream) {
+                                             float softcap, int qkv_ld, cudaStream_t stream) {
+    // rows of the product may go on behind the heads; a layer that writes no keys may have the query heads alone
+    LILY_REQUIRE(qkv_ld % 2 == 0 && qkv_ld >= (write_kv ? nq + 2 * nkv : nq) * d, "attention_decode_fused: rows of %d numbers", qkv_ld);
     LILY_REQUIRE(qkv != nullptr && qkv_planes >= 1 && (qkv_dtype == kF32 || qkv_planes == 1),
                  "attention_decode_fused: %d planes of dtype %d", qkv_planes, qkv_dtype);
     LILY_REQUIRE(rd >= 0 && rd <= d && rd % 2 == 0, "attention_decode_fused: rotary_dim %d does not fit head_dim %d", rd, d);
@@ -938,6 +940,7 @@ LILY_API int lily_attention_decode_mma_fused(const void* qkv, int qkv_planes, si
     a.q_gain = q_gain; a.k_gain = k_gain; a.gain_f32 = gain_dtype == kF32; a.eps = eps;
     a.cos_t = cos_t; a.sin_t = sin_t; a.rd = cos_t ? rd : 0; a.write_kv = write_kv;
     a.softcap = softcap;
+    a.qkv_ld = qkv_ld;
     return decode_mma(a, nullptr, kv, out, block_table, bt_stride, seq_lens, scratch, requests, splits, nq, nkv, d,
                       page_size, window, scale, stages, stream);
 }

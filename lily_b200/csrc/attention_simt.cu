@@ -8,7 +8,8 @@
 // [kv_heads, page_size, dv], and outputs have dv columns a head.  Or the values are the first dv columns of the key
 // rows themselves (`v_in_k`, attention over a cached latent that serves as key and value): a page is then its keys alone.
 // `sink`: a row's running (max, sum) start at (0, 1), a key of score 0 that has no value, so the weights are
-// exp(s_j) / (1 + sum exp(s_j)).  `v_all`: a query head's weights meet the values of every kv head at once (a value row
+// exp(s_j) / (1 + sum exp(s_j)); with `sinks` the key's score is a number of the query head instead (not scaled), and they
+// start at (sink, 1).  `v_all`: a query head's weights meet the values of every kv head at once (a value row
 // of nkv * dv columns gathered from the heads' tiles of the page), for callers that mix the heads' weights afterwards:
 // sum_g T[h][g] (P_g V_c) = (sum_g T[h][g] P_g) V_c.  `v_shift`: instead, a query head of kv head g reads the values of kv head
 // (g + v_shift) % nkv, so that nkv launches give the same sums as planes (more than 512 value columns a row).
@@ -117,7 +118,7 @@ attention_simt_kernel(const AttnArgs a) {
     for (int i = 0; i < RPW; ++i) {
         // the sink counts once a row: in the block of the first key range
         const bool sunk = a.sink && (!DECODE || blockIdx.z == 0);
-        m[i] = sunk ? 0.f : -INFINITY;
+        m[i] = sunk ? (a.sinks ? (row_ok[i] ? a.sinks[row_head[i]] : 0.f) : 0.f) : -INFINITY;
         l[i] = sunk ? 1.f : 0.f;
 #pragma unroll
         for (int c = 0; c < DCH; ++c) acc[i][c] = 0.f;
@@ -376,7 +377,7 @@ LILY_API int lily_attention_prefill_simt(const void* q, const void* kv, void* ou
                                          int bt_stride, const int* cu_seqlens, const int* prefix_lens,
                                          const int* tile_req, const int* tile_start, int tiles, int nq, int nkv,
                                          int d, int page_size, int window, float scale, int dtype,
-                                         float softcap, int dv, int keep_first, int flags, int v_shift, cudaStream_t stream) {
+                                         float softcap, int dv, int keep_first, int flags, int v_shift, const float* sinks, cudaStream_t stream) {
     if (tiles == 0) return 0;
     LILY_REQUIRE(v_shift >= 0 && v_shift < nkv && !(v_shift && dv < 0), "attention_prefill: value heads shifted by %d of %d", v_shift, nkv);
     if (check_common("attention_prefill", nq, nkv, d, page_size, dv)) return 1;
@@ -389,6 +390,8 @@ LILY_API int lily_attention_prefill_simt(const void* q, const void* kv, void* ou
     a.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
     if (apply_flags("attention_prefill", a, flags)) return 1;
     a.v_shift = v_shift;
+    a.sinks = sinks;
+    a.sink = a.sink || sinks != nullptr;
     dim3 grid(tiles, nq);
     int rc = dtype == kBF16 ? launch<__nv_bfloat16, false>(a, grid, stream) : launch<float, false>(a, grid, stream);
     if (rc) return rc;
@@ -423,7 +426,7 @@ LILY_API int lily_attention_decode_simt(const void* q, const void* kv, void* out
                                         int bt_stride, const int* seq_lens, float* scratch, int requests,
                                         int splits, int nq, int nkv, int d, int page_size, int window,
                                         float scale, int dtype, float softcap, int dv, int keep_first, int flags, int v_shift,
-                                        cudaStream_t stream) {
+                                        const float* sinks, cudaStream_t stream) {
     if (requests == 0) return 0;
     LILY_REQUIRE(v_shift >= 0 && v_shift < nkv && !(v_shift && dv < 0), "attention_decode: value heads shifted by %d of %d", v_shift, nkv);
     if (check_common("attention_decode", nq, nkv, d, page_size, dv)) return 1;
@@ -439,6 +442,8 @@ LILY_API int lily_attention_decode_simt(const void* q, const void* kv, void* out
     a.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
     if (apply_flags("attention_decode", a, flags)) return 1;
     a.v_shift = v_shift;
+    a.sinks = sinks;
+    a.sink = a.sink || sinks != nullptr;
     a.part_o = scratch;
     a.part_ml = scratch ? scratch + (size_t)requests * nq * splits * d_out : nullptr;
     dim3 grid(requests, nkv * chunks, splits);

@@ -1,6 +1,7 @@
 // Kernels that join the outputs of sublayers which read the same input:
 //
 //   sigmoid gate:   out[t][c] *= sigmoid(gate[t][c])                    (an output gate ahead of a projection)
+//   head gate:      out[t][h][c] *= sigmoid(gate[t][h])                  (the same with one number a head)
 //   normed mean:    out[t] = scale * sum_k rms(in_k[t]) * gain_k  (+ add[t])      as float32
 //
 //   head mix:       out[t][h][c] = sum_g mix[h][g] * in[t][g][kv(h)][c]                  (attention weights mixed over heads)
@@ -52,6 +53,31 @@ __global__ void sigmoid_gate_bf16x8_kernel(__nv_bfloat16* __restrict__ out, cons
             o2[k] = __floats2bfloat162_rn(__fdividef(o.x, 1.f + __expf(-g.x)), __fdividef(o.y, 1.f + __expf(-g.y)));
         }
         *reinterpret_cast<uint4*>(out + i) = ov;
+    }
+}
+
+// In place, one gate a head: out[t][h][c] *= sigmoid(gate[t * ld + g0 + h]).  VEC neighbouring columns of one head a thread (8
+// in bfloat16, 4 in float32: 16 bytes; 1 when the head's columns do not divide).
+template <typename T, int VEC>
+__global__ void sigmoid_head_gate_kernel(T* __restrict__ out, const Operand gate, int ld, int g0, int heads, int dv, size_t total) {
+    pdl_enter_small();
+    const size_t step = (size_t)gridDim.x * blockDim.x * VEC;
+    for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC; i < total; i += step) {
+        const size_t row = i / dv;                               // token * heads + head
+        const float g = 1.f / (1.f + expf(-gate((row / heads) * ld + g0 + row % heads)));
+        if constexpr (VEC == 8) {
+            uint4 v = *reinterpret_cast<const uint4*>(out + i);
+            __nv_bfloat162* v2 = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const float2 o = __bfloat1622float2(v2[k]);
+                v2[k] = __floats2bfloat162_rn(o.x * g, o.y * g);
+            }
+            *reinterpret_cast<uint4*>(out + i) = v;
+        } else {
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) out[i + k] = from_float<T>(to_float(out[i + k]) * g);
+        }
     }
 }
 
@@ -247,6 +273,25 @@ LILY_API int lily_sigmoid_gate(void* out, int out_dtype, const void* gate, int g
     } else if (out_dtype == kBF16) launch_pdl(sigmoid_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (__nv_bfloat16*)out, g, total);
     else launch_pdl(sigmoid_gate_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)out, g, total);
     LILY_CHECK_LAUNCH("sigmoid_gate");
+    return 0;
+}
+
+LILY_API int lily_sigmoid_head_gate(void* out, int out_dtype, const void* gate, int gate_dtype, int gate_splits, size_t gate_stride, int ld,
+                                    int g0, int tokens, int heads, int dv, cudaStream_t stream) {
+    const size_t total = (size_t)tokens * heads * dv;
+    if (total == 0) return 0;
+    LILY_REQUIRE(heads > 0 && dv > 0 && g0 >= 0 && g0 + heads <= ld, "sigmoid_head_gate: %d heads of %d columns, gates from column %d of %d", heads, dv, g0, ld);
+    LILY_REQUIRE(gate_splits >= 1 && (gate_splits == 1 || gate_dtype == kF32), "sigmoid_head_gate: only float32 partial sums come in several splits");
+    const Operand g{gate, gate_dtype == kBF16, gate_splits, gate_stride};
+    const int most = out_dtype == kBF16 ? 8 : 4;
+    const bool wide = dv % most == 0 && ((uintptr_t)out & 15) == 0;
+    const size_t work = total / (wide ? most : 1);
+    const int blocks = (int)((work + 255) / 256 < (size_t)sm_count() * 16 ? (work + 255) / 256 : (size_t)sm_count() * 16);
+#define GO(T, V) launch_pdl(sigmoid_head_gate_kernel<T, V>, dim3(blocks), dim3(256), 0, stream, (T*)out, g, ld, g0, heads, dv, total)
+    if (out_dtype == kBF16) { if (wide) GO(__nv_bfloat16, 8); else GO(__nv_bfloat16, 1); }
+    else { if (wide) GO(float, 4); else GO(float, 1); }
+#undef GO
+    LILY_CHECK_LAUNCH("sigmoid_head_gate");
     return 0;
 }
 

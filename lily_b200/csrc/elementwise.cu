@@ -359,7 +359,7 @@ __global__ void qk_norm_rope_write_kernel(const Summed<IN> qkv, const W* __restr
                                           const int* __restrict__ positions, const int* __restrict__ token_req,
                                           const int* __restrict__ block_table, int bt_stride,
                                           T* __restrict__ kv_layer, T* __restrict__ q_out,
-                                          int nq, int nkv, int dk, int rd, int page_size, int write_kv, int dv,
+                                          int nq, int nkv, int dk, int rd, int page_size, int write_kv, int dv, int ld,
                                           int v_norm, float v_blend, float* __restrict__ v_first, int v_first_mode) {
     pdl_enter_small();
     const int n = blockIdx.x;
@@ -368,8 +368,8 @@ __global__ void qk_norm_rope_write_kernel(const Summed<IN> qkv, const W* __restr
     if (head >= nheads) return;
     const int lane = threadIdx.x;
     const int pos = positions[n];
-    // a row is [q heads of dk | k heads of dk | v heads of dv]; a page its keys [nkv, page, dk], then its values [nkv, page, dv]
-    size_t src = (size_t)n * ((size_t)(nq + nkv) * dk + (size_t)nkv * dv) + (size_t)head * dk;
+    // a row is [q heads of dk | k heads of dk | v heads of dv | anything], `ld` numbers; a page its keys [nkv, page, dk], then its values [nkv, page, dv]
+    size_t src = (size_t)n * ld + (size_t)head * dk;
     int d = dk;
     T* dst;
     const W* gain = nullptr;
@@ -385,7 +385,7 @@ __global__ void qk_norm_rope_write_kernel(const Summed<IN> qkv, const W* __restr
         const int page = block_table[(size_t)token_req[n] * bt_stride + pos / page_size];
         T* base = kv_layer + (size_t)page * nkv * page_size * (dk + dv);
         if (is_v) {
-            src = (size_t)n * ((size_t)(nq + nkv) * dk + (size_t)nkv * dv) + (size_t)(nq + nkv) * dk + (size_t)kvh * dv;
+            src = (size_t)n * ld + (size_t)(nq + nkv) * dk + (size_t)kvh * dv;
             d = dv;
             dst = base + (size_t)nkv * page_size * dk + ((size_t)kvh * page_size + (pos % page_size)) * dv;
         } else {
@@ -506,7 +506,7 @@ __global__ void qk_norm_rope_write_wide_kernel(const __nv_bfloat16* __restrict__
                                                const int* __restrict__ positions, const int* __restrict__ token_req,
                                                const int* __restrict__ block_table, int bt_stride,
                                                __nv_bfloat16* __restrict__ kv_layer, __nv_bfloat16* __restrict__ q_out,
-                                               int nq, int nkv, int d, int group, int page_size, int write_kv) {
+                                               int nq, int nkv, int d, int group, int page_size, int write_kv, int ld) {
     pdl_enter_small();
     const int n = blockIdx.x;
     const int per_block = blockDim.x / group;
@@ -522,7 +522,7 @@ __global__ void qk_norm_rope_write_wide_kernel(const __nv_bfloat16* __restrict__
     float a[8], b[8];
     uint4 ra = make_uint4(0, 0, 0, 0), rb = ra;
     if (valid) {
-        const __nv_bfloat16* src = qkv + ((size_t)n * (nq + 2 * nkv) + head) * d;
+        const __nv_bfloat16* src = qkv + (size_t)n * ld + (size_t)head * d;
         ra = *reinterpret_cast<const uint4*>(src + 8 * j);
         rb = *reinterpret_cast<const uint4*>(src + half + 8 * j);
         if (head < nq) {
@@ -777,9 +777,10 @@ LILY_API int lily_qk_norm_rope_write(const void* qkv, const void* q_gain, const 
                                      void* q_out, int tokens, int nq, int nkv, int d, int rd, int page_size,
                                      int write_kv, int act_dtype, int gain_dtype, int in_dtype, int splits,
                                      size_t stride, int dv, int v_norm, float v_blend, float* v_first, int v_first_mode,
-                                     cudaStream_t stream) {
+                                     int ld, cudaStream_t stream) {
     if (tokens == 0) return 0;
     if (dv <= 0) dv = d;
+    LILY_REQUIRE(ld >= (write_kv ? (nq + nkv) * d + nkv * dv : nq * d), "qk_norm_rope_write: rows of %d numbers", ld);
     LILY_REQUIRE(v_first_mode >= 0 && v_first_mode <= 2 && (v_first_mode == 0) == (v_first == nullptr),
                  "qk_norm_rope_write: kept values come with mode 1 (write) or 2 (blend)");
     LILY_REQUIRE(d > 0 && rd >= 0 && rd <= d && rd % 2 == 0, "qk_norm_rope_write: rotary_dim %d does not fit head_dim %d", rd, d);
@@ -789,16 +790,16 @@ LILY_API int lily_qk_norm_rope_write(const void* qkv, const void* q_gain, const 
     const int nheads = write_kv ? nq + 2 * nkv : nq;
     dim3 grid(tokens, (nheads + 3) / 4), block(32, 4);
     const int rot = cos_t ? rd : 0;
-    const bool vec = d % 2 == 0 && dv % 2 == 0 && rot % 4 == 0 && stride % 2 == 0 && aligned16(qkv) && aligned16(kv_layer) &&
+    const bool vec = d % 2 == 0 && dv % 2 == 0 && ld % 2 == 0 && rot % 4 == 0 && stride % 2 == 0 && aligned16(qkv) && aligned16(kv_layer) &&
                      aligned16(q_out) && aligned16(q_gain) && aligned16(k_gain) && aligned16(cos_t) && aligned16(sin_t);
 #define LAUNCH_V(T, W, IN, V)                                                                                     \
     launch_pdl(qk_norm_rope_write_kernel<T, W, IN, V>, grid, block, 0, stream, Summed<IN>{(const IN*)qkv, splits, stride}, \
         (const W*)q_gain, (const W*)k_gain, eps, cos_t, sin_t, positions, token_req, block_table, bt_stride,      \
-        (T*)kv_layer, (T*)q_out, nq, nkv, d, rot, page_size, write_kv, dv, v_norm, v_blend, v_first, v_first_mode)
+        (T*)kv_layer, (T*)q_out, nq, nkv, d, rot, page_size, write_kv, dv, ld, v_norm, v_blend, v_first, v_first_mode)
 #define LAUNCH(T, W, IN) do { if (vec) LAUNCH_V(T, W, IN, 2); else LAUNCH_V(T, W, IN, 1); } while (0)
     const bool gb = gain_dtype == kBF16, ib = in_dtype == kBF16;
     const int group = d / 16;
-    if (!v_norm && !v_first_mode && act_dtype == kBF16 && ib && splits == 1 && dv == d && d % 16 == 0 && group <= 32 && (group & (group - 1)) == 0 &&
+    if (!v_norm && !v_first_mode && act_dtype == kBF16 && ib && splits == 1 && dv == d && d % 16 == 0 && ld % 8 == 0 && group <= 32 && (group & (group - 1)) == 0 &&
         (rot == d || rot == 0) && aligned16(qkv) && aligned16(kv_layer) && aligned16(q_out) && aligned16(q_gain) &&
         aligned16(k_gain) && aligned16(cos_t) && aligned16(sin_t)) {
         const int per_block = 128 / group;
@@ -806,11 +807,11 @@ LILY_API int lily_qk_norm_rope_write(const void* qkv, const void* q_gain, const 
         if (gb)
             launch_pdl(qk_norm_rope_write_wide_kernel<__nv_bfloat16>, wgrid, dim3(128), 0, stream, (const __nv_bfloat16*)qkv,
                        (const __nv_bfloat16*)q_gain, (const __nv_bfloat16*)k_gain, eps, cos_t, sin_t, positions, token_req,
-                       block_table, bt_stride, (__nv_bfloat16*)kv_layer, (__nv_bfloat16*)q_out, nq, nkv, d, group, page_size, write_kv);
+                       block_table, bt_stride, (__nv_bfloat16*)kv_layer, (__nv_bfloat16*)q_out, nq, nkv, d, group, page_size, write_kv, ld);
         else
             launch_pdl(qk_norm_rope_write_wide_kernel<float>, wgrid, dim3(128), 0, stream, (const __nv_bfloat16*)qkv,
                        (const float*)q_gain, (const float*)k_gain, eps, cos_t, sin_t, positions, token_req,
-                       block_table, bt_stride, (__nv_bfloat16*)kv_layer, (__nv_bfloat16*)q_out, nq, nkv, d, group, page_size, write_kv);
+                       block_table, bt_stride, (__nv_bfloat16*)kv_layer, (__nv_bfloat16*)q_out, nq, nkv, d, group, page_size, write_kv, ld);
         LILY_CHECK_LAUNCH("qk_norm_rope_write");
         return 0;
     }

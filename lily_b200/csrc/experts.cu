@@ -4,12 +4,14 @@
 //
 //   route     z = W_router h (float32); s = softmax(z) over all router outputs, or sigmoid(z) one by one; the `top`
 //             largest s (+ correction) are chosen; their weights are s, or s / (sum of the chosen s + 1e-20).  One more
-//             row of the matrix may follow the outputs': the sigmoid of its product is the token's gate for a shared expert
+//             row of the matrix may follow the outputs': the sigmoid of its product is the token's gate for a shared expert.
+//             With groups (equal runs of neighbouring outputs) only outputs of the `keep` best groups can be chosen; a
+//             group's score is the sum of its two largest choice scores
 //   align     pairs (token, choice) whose expert has weights are grouped by expert: offsets, the pairs in grouped
 //             order, each pair's place there, and the list of (expert, first row) tiles the products run over
 //   gate/up   a[row, n] = g sigmoid(alpha g) (u + 1), g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit), or
 //             silu(g) u with g = W_gate x, u = W_up x; a weight that belongs to the expert's input multiplies g and u
-//             ahead of the activation (both are linear in x)
+//             ahead of the activation (both are linear in x).  An ungated expert has W_up alone: a = max(W_up x, 0)^2
 //   down      y[row, :] = W_down a[row, :]                                  (float32)
 //   combine   out[t] = sum over the token's choices of weight * (y of the pair, or the token's input itself where the
 //             chosen router output is one of the last `identity` ones, which have no weights); without the weight where
@@ -24,12 +26,29 @@ namespace lily {
 
 constexpr int ROUTE_MAX = 1024;       // router outputs
 constexpr int ROUTE_TOP_MAX = 64;
+constexpr int ROUTE_GROUPS_MAX = 128;
+
+// Groups of router outputs: `count` equal runs of neighbours (0: none), of which the `keep` best can be chosen from.
+struct RouteGroups {
+    int count, keep;
+};
+
+// The two largest of a set, kept while numbers come in.
+struct BestTwo {
+    float first = -INFINITY, second = -INFINITY;
+    __device__ __forceinline__ void add(float v) {
+        if (v > first) { second = first; first = v; }
+        else if (v > second) second = v;
+    }
+    // a set of one number scores that number
+    __device__ __forceinline__ float sum() const { return second > -INFINITY ? first + second : first; }
+};
 
 // Scores and choice of token t by one warp.  s: the token's logits in shared memory (overwritten), `outputs` of them and, with
 // `gate`, the shared gate's behind them; picked: room for `top` numbers.
 __device__ __forceinline__ void choose_experts(float* s, int t, int outputs, const float* __restrict__ correction, int top, int sigmoid,
-                                               int renormalise, float* picked, int* __restrict__ chosen, float* __restrict__ weights,
-                                               float* __restrict__ gate) {
+                                               int renormalise, RouteGroups groups, float* picked, int* __restrict__ chosen,
+                                               float* __restrict__ weights, float* __restrict__ gate) {
     const int lane = threadIdx.x & 31, rows = outputs + (gate ? 1 : 0);
     float inv = 1.f;
     if (sigmoid) {
@@ -53,13 +72,50 @@ __device__ __forceinline__ void choose_experts(float* s, int t, int outputs, con
         if (gate && lane == 0) gate[t] = 1.f / (1.f + expf(-s[outputs]));
     }
     __syncwarp();
+    if (groups.count > 1) {
+        // a lane a group and turn: its score, then its place among the groups (ties: the earlier one); the outputs of the
+        // groups that are not kept are marked as taken
+        const int size = outputs / groups.count;
+        float score[ROUTE_GROUPS_MAX / 32];
+#pragma unroll
+        for (int r = 0; r < ROUTE_GROUPS_MAX / 32; ++r) {
+            const int g = lane + 32 * r;
+            score[r] = -INFINITY;
+            if (g < groups.count) {
+                BestTwo two;
+                for (int e = g * size; e < (g + 1) * size; ++e) two.add(correction ? s[e] * inv + correction[e] : s[e] * inv);
+                score[r] = two.sum();
+            }
+        }
+        int ahead[ROUTE_GROUPS_MAX / 32] = {};
+#pragma unroll
+        for (int r = 0; r < ROUTE_GROUPS_MAX / 32; ++r) {
+            if (32 * r >= groups.count) break;
+            for (int l = 0; l < 32; ++l) {
+                const float other = __shfl_sync(0xffffffffu, score[r], l);
+                const int og = 32 * r + l;
+                if (og >= groups.count) continue;
+#pragma unroll
+                for (int q = 0; q < ROUTE_GROUPS_MAX / 32; ++q)
+                    ahead[q] += other > score[q] || (other == score[q] && og < lane + 32 * q);
+            }
+        }
+        __syncwarp();
+#pragma unroll
+        for (int r = 0; r < ROUTE_GROUPS_MAX / 32; ++r) {
+            const int g = lane + 32 * r;
+            if (g < groups.count && ahead[r] >= groups.keep)
+                for (int e = g * size; e < (g + 1) * size; ++e) s[e] = -1.f;
+        }
+        __syncwarp();
+    }
     float total = 0.f;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int at = outputs;
         for (int e = lane; e < outputs; e += 32) {
             const float p = s[e];
-            if (p < 0.f) continue;                                // taken already
+            if (p < 0.f) continue;                                // taken already, or in a group that is not kept
             const float c = correction ? p * inv + correction[e] : p * inv;
             if (c > best) { best = c; at = e; }
         }
@@ -87,7 +143,7 @@ __device__ __forceinline__ void choose_experts(float* s, int t, int outputs, con
 // The choice from logits that a product has left (finished rows or partial sums).  grid (ceil(tokens / 4)), block 128: a
 // warp a token.
 __global__ void moe_choose_kernel(const Operand logits, int ld, int tokens, const float* __restrict__ correction, int outputs, int top, int sigmoid,
-                                  int renormalise, int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ gate) {
+                                  int renormalise, const RouteGroups groups, int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ gate) {
     __shared__ float picked[4][ROUTE_TOP_MAX];
     extern __shared__ __align__(16) float dyn[];             // [4][rows]
     pdl_enter_small();
@@ -96,7 +152,7 @@ __global__ void moe_choose_kernel(const Operand logits, int ld, int tokens, cons
     float* s = dyn + warp * rows;
     for (int e = lane; e < rows; e += 32) s[e] = logits((size_t)t * ld + e);
     __syncwarp();
-    choose_experts(s, t, outputs, correction, top, sigmoid, renormalise, picked[warp], chosen, weights, gate);
+    choose_experts(s, t, outputs, correction, top, sigmoid, renormalise, groups, picked[warp], chosen, weights, gate);
 }
 
 // grid (ceil(tokens / TB)), block 128: a block takes TB tokens, so a number of the router matrix read once serves TB
@@ -105,7 +161,7 @@ __global__ void moe_choose_kernel(const Operand logits, int ld, int tokens, cons
 template <typename T, int TB>
 __global__ void moe_route_kernel(const T* __restrict__ h, int tokens, int width, const float* __restrict__ router,
                                  const float* __restrict__ correction, int outputs, int top, int sigmoid, int renormalise,
-                                 int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ gate) {
+                                 const RouteGroups groups, int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ gate) {
     __shared__ float picked[4][ROUTE_TOP_MAX];
     extern __shared__ __align__(16) float dyn[];             // [TB][width] the tokens' rows, then [TB][rows of the matrix] their scores
     const int rows = outputs + (gate ? 1 : 0);
@@ -181,7 +237,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int tokens, int width,
     }
     __syncthreads();
     for (int j = warp; j < nt; j += nwarp)
-        choose_experts(sc + j * rows, t0 + j, outputs, correction, top, sigmoid, renormalise, picked[warp], chosen, weights, gate);
+        choose_experts(sc + j * rows, t0 + j, outputs, correction, top, sigmoid, renormalise, groups, picked[warp], chosen, weights, gate);
 }
 
 // One block of 1024 threads.  chosen [pairs]; experts: router outputs that have weights (the rest are skipped here).
@@ -235,7 +291,8 @@ __global__ void moe_align_kernel(const int* __restrict__ chosen, int pairs, int 
 
 // The grouped products.  grid (ceil(N / BN), max_tiles), block 256: tile `blockIdx.y` of the list holds up to BM rows
 // of one expert.  MODE 0: A rows are the tokens of the pairs (pair / top), W = [gate rows | up rows] of the expert,
-// the output is the activation in T.  MODE 1: A rows are the rows of `a` in grouped order, the output float32.
+// the output is the activation in T.  MODE 1: A rows are the rows of `a` in grouped order, the output float32.  MODE 2: as
+// mode 0 for ungated experts, W = the up rows alone.
 constexpr int EBM = 32, EBN = 64, EBK = 16;
 
 // act 0: the clamped gate; 1: silu(g) u
@@ -244,6 +301,11 @@ __device__ __forceinline__ float expert_gate(int act, float g, float u, float li
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return (g / (1.f + expf(-alpha * g))) * (u + 1.f);
+}
+
+__device__ __forceinline__ float squared_relu(float z) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
 }
 
 template <typename T, int MODE>
@@ -263,7 +325,7 @@ moe_gemm_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, size_
     const T* We = W + (size_t)e * w_expert;
     if (threadIdx.x < EBM) {
         const int r = threadIdx.x;
-        arow[r] = r < rows ? (MODE == 0 ? order[row0 + r] / top : row0 + r) : -1;
+        arow[r] = r < rows ? (MODE != 1 ? order[row0 + r] / top : row0 + r) : -1;
     }
     __syncthreads();
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;          // 4 columns, 2 rows a thread
@@ -312,6 +374,9 @@ moe_gemm_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, size_
             if (MODE == 0) {
                 const float w = in_weight ? in_weight[order[row0 + r]] : 1.f;
                 ((T*)out)[(size_t)(row0 + r) * N + n] = from_float<T>(expert_gate(act, w * acc[i][j], w * acc2[i][j], limit, alpha));
+            } else if (MODE == 2) {
+                const float w = in_weight ? in_weight[order[row0 + r]] : 1.f;
+                ((T*)out)[(size_t)(row0 + r) * N + n] = from_float<T>(squared_relu(w * acc[i][j]));
             } else {
                 ((float*)out)[(size_t)(row0 + r) * N + n] = acc[i][j];
             }
@@ -379,6 +444,28 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ h, int width
     for (int c = threadIdx.x; c < width / 8; c += blockDim.x) dst[c] = live ? src[c] : make_uint4(0, 0, 0, 0);
 }
 
+// a[row] = max(u[row], 0)^2 with u[row] = the up product (ff), times the pair's weight first where it belongs to the input.
+__global__ void moe_relu2_kernel(const __nv_bfloat16* __restrict__ u, int ff, __nv_bfloat16* __restrict__ a, const float* __restrict__ in_weight,
+                                 const int* __restrict__ offsets, int experts, const int* __restrict__ order) {
+    pdl_wait();
+    const size_t row = blockIdx.x;
+    const bool live = (int)row < offsets[experts];      // a row of no pair: the next product must not read what was never written
+    const float w = live && in_weight ? in_weight[order[row]] : 1.f;
+    for (int c = threadIdx.x; c < ff / 8; c += blockDim.x) {
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (live) {
+            v = reinterpret_cast<const uint4*>(u + row * ff)[c];
+            __nv_bfloat162* v2 = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const float2 z = __bfloat1622float2(v2[k]);
+                v2[k] = __floats2bfloat162_rn(squared_relu(w * z.x), squared_relu(w * z.y));
+            }
+        }
+        reinterpret_cast<uint4*>(a + row * ff)[c] = v;
+    }
+}
+
 // a[row] = gate(gu[row]) with gu[row] = [gate (ff) | up (ff)], both times the pair's weight first where it belongs to the input.
 __global__ void moe_activation_kernel(const __nv_bfloat16* __restrict__ gu, int ff, __nv_bfloat16* __restrict__ a, int act, float limit,
                                       float alpha, const float* __restrict__ in_weight, const int* __restrict__ offsets,
@@ -411,13 +498,22 @@ __global__ void moe_activation_kernel(const __nv_bfloat16* __restrict__ gu, int 
 using namespace lily;
 
 // router [outputs (+ 1 with `gate`), width]; correction [outputs] or null; sigmoid 0: softmax over the outputs, 1: each
-// output's sigmoid; renormalise: the chosen scores over their sum.
+// output's sigmoid; renormalise: the chosen scores over their sum; groups (0 or 1: none) and how many of them are kept.
+static int check_groups(const char* name, int outputs, int top, int groups, int keep) {
+    LILY_REQUIRE(groups >= 0 && groups <= ROUTE_GROUPS_MAX, "%s: %d groups (up to %d)", name, groups, ROUTE_GROUPS_MAX);
+    LILY_REQUIRE(groups <= 1 || (outputs % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (outputs / groups)),
+                 "%s: top %d of the best %d of %d groups of %d outputs", name, top, keep, groups, outputs);
+    return 0;
+}
+
 LILY_API int lily_moe_route(const void* h, int tokens, int width, const float* router, const float* correction, int outputs,
-                            int top, int sigmoid, int renormalise, int* chosen, float* weights, float* gate, int dtype,
+                            int top, int sigmoid, int renormalise, int group_count, int group_keep, int* chosen, float* weights, float* gate, int dtype,
                             cudaStream_t stream) {
     if (tokens == 0) return 0;
     LILY_REQUIRE(outputs >= 1 && outputs <= ROUTE_MAX, "moe_route: %d router outputs (up to %d)", outputs, ROUTE_MAX);
     LILY_REQUIRE(top >= 1 && top <= outputs && top <= ROUTE_TOP_MAX, "moe_route: top %d of %d", top, outputs);
+    if (check_groups("moe_route", outputs, top, group_count, group_keep)) return 1;
+    const RouteGroups groups{group_count, group_keep};
     const int rows = outputs + (gate ? 1 : 0);
     // four tokens a block once there are blocks enough for the device, and while their rows fit the shared memory
     const int tb = (tokens >= 1024 && (size_t)(4 * width + 4 * rows) * sizeof(float) <= 40 * 1024) ? 4 : 1;
@@ -426,7 +522,7 @@ LILY_API int lily_moe_route(const void* h, int tokens, int width, const float* r
     dim3 grid((tokens + tb - 1) / tb), block(128);
 #define GO(T, TB)                                                                                                   \
     launch_pdl(moe_route_kernel<T, TB>, grid, block, smem, stream, (const T*)h, tokens, width, router, correction, outputs, \
-               top, sigmoid, renormalise, chosen, weights, gate)
+               top, sigmoid, renormalise, groups, chosen, weights, gate)
     if (dtype == kBF16) { if (tb == 4) GO(__nv_bfloat16, 4); else GO(__nv_bfloat16, 1); }
     else { if (tb == 4) GO(float, 4); else GO(float, 1); }
 #undef GO
@@ -436,14 +532,16 @@ LILY_API int lily_moe_route(const void* h, int tokens, int width, const float* r
 
 // The same from the logits: rows `ld` apart, outputs (+ 1 with `gate`) of them read.
 LILY_API int lily_moe_choose(const void* logits, int logits_dtype, int splits, size_t stride, int ld, int tokens, const float* correction, int outputs,
-                             int top, int sigmoid, int renormalise, int* chosen, float* weights, float* gate, cudaStream_t stream) {
+                             int top, int sigmoid, int renormalise, int group_count, int group_keep, int* chosen, float* weights, float* gate, cudaStream_t stream) {
     if (tokens == 0) return 0;
     LILY_REQUIRE(outputs >= 1 && outputs <= ROUTE_MAX, "moe_choose: %d router outputs (up to %d)", outputs, ROUTE_MAX);
     LILY_REQUIRE(top >= 1 && top <= outputs && top <= ROUTE_TOP_MAX, "moe_choose: top %d of %d", top, outputs);
     LILY_REQUIRE(splits >= 1 && logits_dtype == kF32 && ld >= outputs + (gate ? 1 : 0), "moe_choose: float32 logits in rows of %d", ld);
+    if (check_groups("moe_choose", outputs, top, group_count, group_keep)) return 1;
+    const RouteGroups groups{group_count, group_keep};
     const Operand x{logits, 0, splits, stride};
     launch_pdl(moe_choose_kernel, dim3((tokens + 3) / 4), dim3(128), (size_t)4 * (outputs + 1) * sizeof(float), stream, x, ld, tokens, correction,
-               outputs, top, sigmoid, renormalise, chosen, weights, gate);
+               outputs, top, sigmoid, renormalise, groups, chosen, weights, gate);
     LILY_CHECK_LAUNCH("moe_choose");
     return 0;
 }
@@ -461,21 +559,22 @@ LILY_API int lily_moe_align(const int* chosen, int pairs, int experts, int* offs
 }
 
 // mode 0: gate/up with the activation (W [experts, 2 N, K], out [pairs, N] in the activation dtype; in_weight: the pairs'
-// weights where they belong to the input, else null); mode 1: down (W [experts, N, K], out [pairs, N] float32).
+// weights where they belong to the input, else null); mode 1: down (W [experts, N, K], out [pairs, N] float32); mode 2: up with
+// the squared relu (W [experts, N, K], out and in_weight as in mode 0).
 LILY_API int lily_moe_gemm(int mode, const void* A, int lda, const void* W, int N, int K, const int* offsets,
                            const int* order, int top, const int* tile_expert, const int* tile_row, const int* tile_count,
                            int max_tiles, void* out, int act, float limit, float alpha, const float* in_weight, int dtype,
                            cudaStream_t stream) {
     if (max_tiles == 0 || N == 0) return 0;
-    LILY_REQUIRE(K > 0 && lda >= K && (mode == 0 || mode == 1), "moe_gemm: mode=%d N=%d K=%d lda=%d", mode, N, K, lda);
+    LILY_REQUIRE(K > 0 && lda >= K && mode >= 0 && mode <= 2, "moe_gemm: mode=%d N=%d K=%d lda=%d", mode, N, K, lda);
     LILY_REQUIRE(max_tiles <= 65535, "moe_gemm: %d tiles", max_tiles);
     dim3 grid((N + EBN - 1) / EBN, max_tiles), block(256);
     const size_t w_expert = (size_t)(mode == 0 ? 2 : 1) * N * K;
 #define GO(T, MODE)                                                                                                \
     launch_pdl(moe_gemm_kernel<T, MODE>, grid, block, 0, stream, (const T*)A, lda, (const T*)W, w_expert, N, K, offsets, \
                order, top, tile_expert, tile_row, tile_count, out, act, limit, alpha, in_weight)
-    if (dtype == kBF16) { if (mode == 0) GO(__nv_bfloat16, 0); else GO(__nv_bfloat16, 1); }
-    else { if (mode == 0) GO(float, 0); else GO(float, 1); }
+    if (dtype == kBF16) { if (mode == 0) GO(__nv_bfloat16, 0); else if (mode == 2) GO(__nv_bfloat16, 2); else GO(__nv_bfloat16, 1); }
+    else { if (mode == 0) GO(float, 0); else if (mode == 2) GO(float, 2); else GO(float, 1); }
 #undef GO
     LILY_CHECK_LAUNCH("moe_gemm");
     return 0;
@@ -522,5 +621,16 @@ LILY_API int lily_moe_activation(const void* gu, int ff, int rows, void* a, int 
     launch_pdl(moe_activation_kernel, dim3(rows), dim3(ff >= 1024 ? 128 : (ff >= 512 ? 64 : 32)), 0, stream, (const __nv_bfloat16*)gu, ff,
                (__nv_bfloat16*)a, act, limit, alpha, in_weight, offsets, experts, order);
     LILY_CHECK_LAUNCH("moe_activation");
+    return 0;
+}
+
+// The same for ungated experts: u [rows, ff] the up product, a = max(u, 0)^2.
+LILY_API int lily_moe_relu2(const void* u, int ff, int rows, void* a, const float* in_weight, const int* offsets, int experts, const int* order,
+                            cudaStream_t stream) {
+    if (rows == 0) return 0;
+    LILY_REQUIRE(ff % 8 == 0 && ((uintptr_t)u & 15) == 0 && ((uintptr_t)a & 15) == 0, "moe_relu2: rows of %d are not whole 16-byte pieces", ff);
+    launch_pdl(moe_relu2_kernel, dim3(rows), dim3(ff >= 1024 ? 128 : (ff >= 512 ? 64 : 32)), 0, stream, (const __nv_bfloat16*)u, ff,
+               (__nv_bfloat16*)a, in_weight, offsets, experts, order);
+    LILY_CHECK_LAUNCH("moe_relu2");
     return 0;
 }

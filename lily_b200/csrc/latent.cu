@@ -6,7 +6,7 @@
 // the head's output is W_uv (sum_j p_j latent_j): the attention kernel runs over the rows as they are cached, all
 // heads sharing them, and reads its values out of the first `rank` columns of the key rows.
 //
-//   latent_prepare  down-projection row -> RMS-normed query latent; RMS-normed key/value latent and the rotated
+//   latent_prepare  down-projection row -> RMS-normed query latent (none when the queries have no latent of their own); RMS-normed key/value latent and the rotated
 //                   key part into the token's cache row
 //   latent_query    the rotated part of every head's query, beside the part the per-head product has put in place
 //   head_gate       per-head outputs times sigmoid(gate of the head) -> the rows the output projection takes
@@ -80,7 +80,7 @@ __global__ void latent_prepare_kernel(const Operand in, int ld, int q0, int q_ra
         ssq += sums[0][w];
         ssk += sums[1][w];
     }
-    const float inv_q = rsqrtf(ssq / (float)q_rank + eps);
+    const float inv_q = rsqrtf(ssq / (float)max(q_rank, 1) + eps);
     if (VEC == 4)
         for (int c = threadIdx.x * 4; c < q_rank; c += blockDim.x * 4) {
             const float4 x = *reinterpret_cast<const float4*>(held + c), g = *reinterpret_cast<const float4*>(q_gain + c);
@@ -176,7 +176,7 @@ LILY_API int lily_latent_prepare(const void* in, int in_dtype, int in_splits, si
                                  const int* block_table, int bt_stride, void* layer, int page_size, int write_kv, void* cq,
                                  int tokens, int dtype, cudaStream_t stream) {
     if (tokens == 0) return 0;
-    LILY_REQUIRE(q_rank > 0 && rank > 0 && rot >= 0 && rd >= 0 && rd <= rot && rd % 2 == 0,
+    LILY_REQUIRE(q_rank >= 0 && rank > 0 && rot >= 0 && rd >= 0 && rd <= rot && rd % 2 == 0,
                  "latent_prepare: q_rank=%d rank=%d rot=%d rotated=%d", q_rank, rank, rot, rd);
     LILY_REQUIRE(rd == 0 || !write_kv || (cos_t && sin_t), "latent_prepare: rotation needs its tables");
     LILY_REQUIRE(in_splits >= 1 && (in_splits == 1 || in_dtype == kF32), "latent_prepare: only float32 partial sums come in several splits");

@@ -16,6 +16,9 @@
 // whose (max, sum, output) go to scratch in the layout the combine kernel merges
 // (lily_attention_combine: [requests, heads, ranges, rank] outputs, then [.., 2]).
 //
+// With `sinks` a row's running (max, sum) start at (the head's sink, 1): the softmax's denominator holds exp(sink), a key
+// without a value whose score is not scaled (decode: in the first key range).
+//
 // Scores, softmax and sums are float32; the weights are rounded to bfloat16 for their product with the values.
 // The wait for a tile is bounded: when it runs out the block records it in a status word (lily_latent_attention_status),
 // gives the copies it still has in flight a bounded wait and returns.
@@ -85,6 +88,7 @@ struct Args {
     float* part_o;                // decode with ranges
     float* part_ml;
     int splits, heads, row, rank, page_size, window, tile_tokens;
+    const float* sinks;           // [heads], or null
     int rowp;                     // bfloat16 per row of the query and key tiles in shared memory
     float scale;
 };
@@ -188,6 +192,11 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_kernel(const Args
 
     const float sl2 = a.scale * 1.4426950408889634f;
     float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
+    if (a.sinks && (!DECODE || blockIdx.z == 0)) {                  // maxima are in log2 units
+        m_lo = a.sinks[gr_lo % a.heads] * 1.4426950408889634f;
+        m_hi = a.sinks[gr_hi % a.heads] * 1.4426950408889634f;
+        l_lo = l_hi = 1.f;
+    }
     float o[VT][4];
 #pragma unroll
     for (int j = 0; j < VT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
@@ -428,7 +437,7 @@ LILY_API int lily_latent_attention_prefill_mma(const void* q, const void* cache,
                                                int bt_stride, const int* cu_seqlens, const int* prefix_lens,
                                                const int* tile_req, const int* tile_start, int tiles, int tile_tokens,
                                                int heads, int row, int rank, int page_size, int window, float scale,
-                                               cudaStream_t stream) {
+                                               const float* sinks, cudaStream_t stream) {
     if (tiles == 0) return 0;
     LILY_REQUIRE(lily_latent_attention_mma_takes(row, rank), "latent attention: rows of %d with rank %d are not for this kernel", row, rank);
     LILY_REQUIRE(heads > 0 && tile_tokens > 0 && page_size > 0, "latent attention: heads=%d tile=%d page=%d", heads, tile_tokens, page_size);
@@ -436,7 +445,7 @@ LILY_API int lily_latent_attention_prefill_mma(const void* q, const void* cache,
     a.q = (const __nv_bfloat16*)q; a.cache = (const __nv_bfloat16*)cache; a.out = (__nv_bfloat16*)out;
     a.block_table = block_table; a.bt_stride = bt_stride; a.cu_seqlens = cu_seqlens; a.prefix_lens = prefix_lens;
     a.tile_req = tile_req; a.tile_start = tile_start; a.splits = 1; a.heads = heads; a.row = row; a.rank = rank;
-    a.page_size = page_size; a.window = window; a.tile_tokens = tile_tokens; a.rowp = row_stride(row, rank); a.scale = scale;
+    a.page_size = page_size; a.window = window; a.tile_tokens = tile_tokens; a.rowp = row_stride(row, rank); a.scale = scale; a.sinks = sinks;
     dim3 grid(tiles, (tile_tokens * heads + ROWS - 1) / ROWS);
     LILY_REQUIRE(grid.y <= 65535, "latent attention: %d heads", heads);
     if (int rc = launch<false>(a, grid, stream)) return rc;
@@ -447,7 +456,7 @@ LILY_API int lily_latent_attention_prefill_mma(const void* q, const void* cache,
 LILY_API int lily_latent_attention_decode_mma(const void* q, const void* cache, void* out, const int* block_table,
                                               int bt_stride, const int* seq_lens, float* scratch, int requests, int splits,
                                               int heads, int row, int rank, int page_size, int window, float scale,
-                                              cudaStream_t stream) {
+                                              const float* sinks, cudaStream_t stream) {
     if (requests == 0) return 0;
     LILY_REQUIRE(lily_latent_attention_mma_takes(row, rank), "latent attention: rows of %d with rank %d are not for this kernel", row, rank);
     LILY_REQUIRE(splits >= 1 && splits <= 65535 && (splits == 1 || scratch), "latent attention: %d key ranges need scratch", splits);
@@ -455,7 +464,7 @@ LILY_API int lily_latent_attention_decode_mma(const void* q, const void* cache, 
     a.q = (const __nv_bfloat16*)q; a.cache = (const __nv_bfloat16*)cache; a.out = (__nv_bfloat16*)out;
     a.block_table = block_table; a.bt_stride = bt_stride; a.seq_lens = seq_lens; a.splits = splits; a.heads = heads;
     a.row = row; a.rank = rank; a.page_size = page_size; a.window = window; a.tile_tokens = 1;
-    a.rowp = row_stride(row, rank); a.scale = scale;
+    a.rowp = row_stride(row, rank); a.scale = scale; a.sinks = sinks;
     a.part_o = scratch;
     a.part_ml = scratch ? scratch + (size_t)requests * heads * splits * rank : nullptr;
     dim3 grid(requests, (heads + ROWS - 1) / ROWS, splits);

@@ -23,6 +23,9 @@
 // (lily_attention_combine: [requests, heads, ranges, rank] outputs, then [.., 2]).  Fewer than 128 heads leave rows of
 // the products unused (their time is the tensor cores' for 128 rows whatever the heads).
 //
+// With `sinks` a row's running maximum starts at the head's sink (in the units of the unscaled scores) and its sum at one:
+// the softmax's denominator holds exp(sink), a key without a value (decode: in the first key range).
+//
 // Keys past the last one a block sees and rows past the tile's are computed on whatever the pages and the neighbouring
 // query rows hold (finite everywhere) and masked, or not stored.  Every wait is bounded; one that runs out sets a status
 // word (lily_latent_attention_tc_status), the roles leave their loops, copies in flight get a bounded wait and the block
@@ -66,6 +69,7 @@ struct Params {
     int col_blocks, cols;                 // column blocks and value columns of one (a multiple of 16)
     int stages, q_rows;                   // rows of the queries' box
     float scale_log2;
+    const float* sinks;                   // [heads], or null
 };
 
 __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatile int* abort_flag, int code) {
@@ -300,6 +304,8 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
         const int pieces = (p.cols + 31) / 32;
         const bool idle = (warp & 3) * 32 >= rows_valid;
         float m_used = -INFINITY, l = 0.f;
+        const bool sunk = p.sinks != nullptr && range == 0;
+        if (sunk) m_used = p.sinks[(row0 + row) % p.heads] * (1.4426950408889634f / p.scale_log2);
         bool ok = true;
         for (int j = 0; j < n && ok; ++j) {
             const int b = j & 1;
@@ -326,6 +332,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
             for (int e = 4; e < BKV; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], s[e]);
             const float m_new = fmaxf(m_used, fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])));
             if (j == 0) {
+                if (sunk) l = ex2((m_used - m_new) * p.scale_log2);
                 m_used = m_new;
             } else {
                 const bool grow = (m_new - m_used) * p.scale_log2 > GROW_LOG2;      // also when m_used is -inf
@@ -500,13 +507,13 @@ static int launch(Params& p, long units, const void* q, const void* cache, int t
 LILY_API int lily_latent_attention_prefill_tc(const void* q, const void* cache, void* out, const int* block_table, int bt_stride,
                                               const int* cu_seqlens, const int* prefix_lens, const int* tile_req, const int* tile_start,
                                               int tiles, int tile_tokens, int heads, int row, int rank, int page_size, int window,
-                                              float scale, int tokens, int num_pages, cudaStream_t stream) {
+                                              float scale, int tokens, int num_pages, const float* sinks, cudaStream_t stream) {
     if (tiles == 0) return 0;
     LILY_REQUIRE(tile_tokens > 0 && (tile_tokens == 1 || tile_tokens * heads <= lt::BQ), "latent_attention_tc: tiles of %d tokens of %d heads", tile_tokens, heads);
     lt::Params p{};
     p.block_table = block_table; p.cu_seqlens = cu_seqlens; p.prefix_lens = prefix_lens; p.tile_req = tile_req; p.tile_start = tile_start;
     p.out = (__nv_bfloat16*)out; p.bt_stride = bt_stride; p.tiles = tiles; p.tile_tokens = tile_tokens; p.heads = heads; p.row = row;
-    p.rank = rank; p.page_size = page_size; p.window = window; p.splits = 1;
+    p.rank = rank; p.page_size = page_size; p.window = window; p.splits = 1; p.sinks = sinks;
     return lt::launch(p, tiles, q, cache, tokens, num_pages, scale, stream);
 }
 
@@ -514,12 +521,12 @@ LILY_API int lily_latent_attention_prefill_tc(const void* q, const void* cache, 
 // results go to scratch, ahead of lily_attention_combine.
 LILY_API int lily_latent_attention_decode_tc(const void* q, const void* cache, void* out, const int* block_table, int bt_stride,
                                              const int* seq_lens, float* scratch, int requests, int splits, int heads, int row, int rank,
-                                             int page_size, int window, float scale, int num_pages, cudaStream_t stream) {
+                                             int page_size, int window, float scale, int num_pages, const float* sinks, cudaStream_t stream) {
     if (requests == 0) return 0;
     LILY_REQUIRE(seq_lens && splits >= 1 && (splits == 1 || scratch), "latent_attention_tc: %d key ranges need scratch", splits);
     lt::Params p{};
     p.block_table = block_table; p.seq_lens = seq_lens; p.splits = splits; p.out = (__nv_bfloat16*)out; p.bt_stride = bt_stride;
-    p.tiles = requests; p.tile_tokens = 1; p.heads = heads; p.row = row; p.rank = rank; p.page_size = page_size; p.window = window;
+    p.tiles = requests; p.tile_tokens = 1; p.heads = heads; p.row = row; p.rank = rank; p.page_size = page_size; p.window = window; p.sinks = sinks;
     p.part_o = splits > 1 ? scratch : nullptr;
     p.part_ml = splits > 1 ? scratch + (size_t)requests * heads * splits * rank : nullptr;
     return lt::launch(p, (long)requests * splits, q, cache, requests, num_pages, scale, stream);

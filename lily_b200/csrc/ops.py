@@ -30,20 +30,25 @@ _SIGNATURES = {
     "lily_silu_mul": [_vp, _vp, _i, _i, _i, _i, _i, _i, _sz, _i, _f, _f, _vp],
     "lily_gemm_tc": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _vp],
     "lily_qk_norm_rope_write": [_vp, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i,
-                                _i, _i, _i, _i, _i, _sz, _i, _i, _f, _vp, _i, _vp],
+                                _i, _i, _i, _i, _i, _sz, _i, _i, _f, _vp, _i, _i, _vp],
     "lily_skinny_gemm": [_vp, _vp, _vp, _i, _i, _i, _i, _vp],
     "lily_skinny_swiglu": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _vp],
     "lily_cast": [_vp, _i, _vp, _i, _sz, _vp],
     "lily_gemm_fp32": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
-    "lily_attention_prefill_simt": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _i, _i, _i, _vp],
-    "lily_attention_decode_simt": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _i, _i, _i, _vp],
+    "lily_attention_prefill_simt": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _i, _i, _i, _vp, _vp],
+    "lily_attention_decode_simt": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _i, _i, _i, _vp, _vp],
     "lily_attention_combine": [_vp, _vp, _i, _i, _i, _i, _i, _vp],
     "lily_attention_prefill_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp],
     "lily_attention_prefill_tc": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _f, _i, _vp],
     "lily_attention_decode_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _i, _i, _vp],
     "lily_attention_decode_mma_fused": [_vp, _i, _sz, _i, _vp, _vp, _i, _f, _vp, _vp, _i, _i, _vp, _vp, _vp, _i, _vp, _vp,
-                                        _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _vp],
+                                        _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _vp],
     "lily_sigmoid_gate": [_vp, _i, _vp, _i, _i, _sz, _sz, _vp],
+    "lily_sigmoid_head_gate": [_vp, _i, _vp, _i, _i, _sz, _i, _i, _i, _i, _i, _vp],
+    "lily_add_tanh_norm": [_vp, _vp, _i, _i, _sz, _f, _vp, _vp, _f, _f, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _vp],
+    "lily_mlstm_scan": [_vp, _i, _i, _sz, _i, _i, _i, _i, _vp, _i, _i, _sz, _i, _i, _i, _vp, _vp, _f, _f, _vp, _sz, _vp, _vp, _vp, _vp, _vp,
+                        _vp, _i, _i, _i, _i, _vp],
+    "lily_mlstm_out": [_vp, _vp, _vp, _vp, _i, _i, _sz, _i, _i, _vp, _f, _f, _vp, _i, _vp, _sz, _sz, _vp, _vp, _vp, _i, _i, _i, _vp],
     "lily_normed_mean": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _sz, _vp, _i, _i, _f, _f, _vp],
     "lily_causal_conv_silu": [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _sz, _sz, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _vp],
     "lily_causal_conv": [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _sz, _sz, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _vp],
@@ -59,10 +64,10 @@ _SIGNATURES = {
                       _i, _vp, _vp, _i, _vp],
     "lily_ssd_combine": [_vp, _sz, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "lily_gated_group_rmsnorm": [_vp, _vp, _i, _vp, _vp, _i, _i, _i, _f, _i, _vp],
-    "lily_latent_attention_prefill_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
-    "lily_latent_attention_prefill_tc": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp],
-    "lily_latent_attention_decode_tc": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
-    "lily_latent_attention_decode_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
+    "lily_latent_attention_prefill_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp],
+    "lily_latent_attention_prefill_tc": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp],
+    "lily_latent_attention_decode_tc": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp],
+    "lily_latent_attention_decode_mma": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp],
     "lily_add_rmsnorm_multi": [_vp, _vp, _i, _i, _sz, _vp, _i, _i, _sz, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _i, _vp],
     "lily_gemm_fp32_heads": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _sz, _sz, _sz, _vp],
     "lily_token_shift_mix": [_vp, _i, _i, _vp, _i, _vp, _sz, _sz, _vp, _vp, _vp, _vp, _i, _vp],
@@ -74,13 +79,14 @@ _SIGNATURES = {
                             _i, _i, _vp],
     "lily_latent_query": [_vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _vp],
     "lily_head_gate": [_vp, _i, _vp, _i, _i, _sz, _i, _i, _i, _i, _i, _vp, _i, _vp],
-    "lily_moe_route": [_vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp],
-    "lily_moe_choose": [_vp, _i, _i, _sz, _i, _i, _vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp],
+    "lily_moe_route": [_vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp],
+    "lily_moe_choose": [_vp, _i, _i, _sz, _i, _i, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp],
     "lily_moe_align": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp],
     "lily_moe_gemm": [_i, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _i, _f, _f, _vp, _i, _vp],
     "lily_moe_combine": [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _i, _sz, _vp, _vp, _i, _vp],
     "lily_moe_gather": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp],
     "lily_moe_activation": [_vp, _i, _i, _vp, _i, _f, _f, _vp, _vp, _i, _vp, _vp],
+    "lily_moe_relu2": [_vp, _i, _i, _vp, _vp, _vp, _i, _vp, _vp],
     "lily_argmax": [_vp, _vp, _vp, _vp, _i, _i, _vp],
     "lily_apply_penalties": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _vp],
     "lily_top_logprobs": [_vp, _vp, _vp, _vp, _vp, _i, _i, _vp],
@@ -137,6 +143,7 @@ def library():
         lib.lily_moe_tile_rows.restype = _i
         lib.lily_delta_rule_max_head_dim.restype = _i
         lib.lily_selective_scan_max_state.restype = _i
+        lib.lily_mlstm_max_head_dim.restype = _i
         _lib = lib
     return _lib
 
@@ -330,18 +337,21 @@ def qk_norm_rope_write(qkv: torch.Tensor, q_gain: Optional[torch.Tensor], k_gain
                        positions: torch.Tensor, token_req: torch.Tensor, block_table: torch.Tensor,
                        kv_layer: torch.Tensor, nq: int, nkv: int, d: int, rotary_dim: int, page_size: int,
                        write_kv: bool = True, q_out: Optional[torch.Tensor] = None, dv: Optional[int] = None,
-                       v_norm: bool = False, v_keep: Optional[torch.Tensor] = None, v_blend: Optional[float] = None) -> torch.Tensor:
+                       v_norm: bool = False, v_keep: Optional[torch.Tensor] = None, v_blend: Optional[float] = None,
+                       row: Optional[int] = None) -> torch.Tensor:
     """Per-head RMSNorm of q and k (when gains are given), rotation by the tables, q to ``q_out``
     [tokens, nq * d], k and v into the token's place in its page of ``kv_layer``.  ``qkv`` is
     [tokens, (nq + nkv) d + nkv dv] in the cache's dtype or float32 partial sums [splits, tokens, ...]; value
     heads have ``dv`` features (default d; see ``cache_layer_fits`` for the page layout).
     ``v_norm``: each value head is divided by its root mean square (``eps``, no gain) before it is cached.
     ``v_keep`` float32 [tokens, nkv * dv]: without ``v_blend`` the (normed) values are also left there; with it they
-    are read from there and the cached value is ``(1 - v_blend) v + v_blend v_keep``."""
+    are read from there and the cached value is ``(1 - v_blend) v + v_blend v_keep``.
+    ``row``: the columns of ``qkv`` where its rows go on behind the heads; without ``write_kv`` they may hold the query heads alone."""
     _dev(qkv, q_gain, k_gain, cos, sin, positions, token_req, block_table, kv_layer, q_out)
     n = qkv.shape[-2]
     dv = int(dv or d)
-    splits, stride = _summed(qkv, n, (nq + nkv) * d + nkv * dv, "qk_norm_rope_write qkv")
+    ld = int(row or (nq + nkv) * d + nkv * dv)
+    splits, stride = _summed(qkv, n, ld, "qk_norm_rope_write qkv")
     if qkv.dtype not in (kv_layer.dtype, torch.float32):
         raise KernelError(f"cache dtype {kv_layer.dtype} differs from activations {qkv.dtype}")
     cache_layer_fits(kv_layer, nkv, page_size, d, dv)
@@ -360,7 +370,7 @@ def qk_norm_rope_write(qkv: torch.Tensor, q_gain: Optional[torch.Tensor], k_gain
           _i32(positions, "positions"), _i32(token_req, "token_req"), _i32(block_table, "block_table"),
           block_table.shape[-1], _p(kv_layer), _p(q_out), n, nq, nkv, d, rotary_dim, page_size, int(write_kv),
           _dt(kv_layer), _dt(q_gain) if q_gain is not None else _F32, _dt(qkv), splits, stride, dv,
-          int(bool(v_norm)), float(v_blend or 0.0), _p(v_keep), 0 if v_keep is None else (1 if v_blend is None else 2), _stream())
+          int(bool(v_norm)), float(v_blend or 0.0), _p(v_keep), 0 if v_keep is None else (1 if v_blend is None else 2), ld, _stream())
     return q_out
 
 
@@ -638,8 +648,10 @@ def attention_prefill(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torc
                       nq: int, nkv: int, d: int, page_size: int, scale: float, window: Optional[int] = None,
                       tile_rows: Optional[int] = None, heads_per_block: int = 0, softcap: Optional[float] = None,
                       dv: Optional[int] = None, values_in_keys: bool = False, keep_first: int = 0,
-                      sink: bool = False, all_values: bool = False) -> None:
+                      sink: bool = False, all_values: bool = False, sinks: Optional[torch.Tensor] = None) -> None:
     """Causal attention of each request's new tokens over its cached prefix and themselves.
+    ``sinks`` (float32, one number a query head): the softmax's denominator holds exp(sinks[h]) as well, a key without a
+    value whose score is not scaled (the kernels over cached latents and the CUDA-core kernel).
     ``sink``: the softmax's denominator holds one more unit (a key of score 0 that has no value).  ``all_values``: every
     query head's weights meet the values of all kv heads, ``out`` is float32 [tokens, nq * nkv * dv] (``head_mix``
     follows).  Both run on the CUDA-core kernel.  ``softcap``: scores
@@ -651,7 +663,8 @@ def attention_prefill(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torc
     in steps of ``tile_rows`` (default: ``prefill_tile_rows(q.dtype, d)``), which also names the
     kernel: the tcgen05 kernel takes tiles of its own size, the others theirs.  ``heads_per_block``
     (tcgen05 only) 1 or 2 picks between its one-head and its two-head form; 0 lets the launcher choose."""
-    _dev(q, kv_layer, block_table, cu_seqlens, prefix_lens, tile_req, tile_start, out)
+    _dev(q, kv_layer, block_table, cu_seqlens, prefix_lens, tile_req, tile_start, out, sinks)
+    _check_sinks(sinks, nq, sink or all_values)
     planes = all_values and out.dim() == 3            # one launch of the mma.sync kernel a kv head (``all_values_sums``)
     if q.dtype != kv_layer.dtype or out.dtype != (torch.float32 if all_values and not planes else q.dtype):
         raise KernelError("attention: q, cache and out must share a dtype (sums over all kv heads' values on CUDA cores are float32)")
@@ -677,7 +690,7 @@ def attention_prefill(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torc
             _call("lily_attention_prefill_simt", _p(q), _p(kv_layer), out[shift].data_ptr(), _i32(block_table, "block_table"),
                   block_table.shape[-1], _i32(cu_seqlens, "cu_seqlens"), _i32(prefix_lens, "prefix_lens"), _i32(tile_req, "tile_req"),
                   _i32(tile_start, "tile_start"), tile_req.numel(), nq, nkv, d, page_size, int(window or 0), float(scale), _dt(q),
-                  float(softcap or 0.0), int(dv or d), int(keep_first or 0) if window else 0, 1 if sink else 0, shift, _stream())
+                  float(softcap or 0.0), int(dv or d), int(keep_first or 0) if window else 0, 1 if sink else 0, shift, None, _stream())
         return
     common = (_p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"), block_table.shape[-1],
               _i32(cu_seqlens, "cu_seqlens"), _i32(prefix_lens, "prefix_lens"), _i32(tile_req, "tile_req"),
@@ -690,21 +703,21 @@ def attention_prefill(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torc
         _call("lily_latent_attention_prefill_tc", _p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"),
               block_table.shape[-1], _i32(cu_seqlens, "cu_seqlens"), _i32(prefix_lens, "prefix_lens"),
               _i32(tile_req, "tile_req"), _i32(tile_start, "tile_start"), tile_req.numel(), int(tile_rows), nq, d, dv,
-              page_size, int(window or 0), float(scale), q.shape[0], kv_layer.shape[0], _stream())
+              page_size, int(window or 0), float(scale), q.shape[0], kv_layer.shape[0], _p(sinks), _stream())
         return
     if (values_in_keys and latent_tensor_cores(q.dtype, d, dv, nkv, softcap)
             and tile_rows == int(lib.lily_latent_attention_mma_tile_tokens(int(nq)))):
         _call("lily_latent_attention_prefill_mma", _p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"),
               block_table.shape[-1], _i32(cu_seqlens, "cu_seqlens"), _i32(prefix_lens, "prefix_lens"),
               _i32(tile_req, "tile_req"), _i32(tile_start, "tile_start"), tile_req.numel(), int(tile_rows), nq, d, dv,
-              page_size, int(window or 0), float(scale), _stream())
+              page_size, int(window or 0), float(scale), _p(sinks), _stream())
         return
     keep_first = int(keep_first or 0) if window else 0
     flags = _attention_flags(sink, all_values, values_in_keys, nkv, dv, out, q.shape[0] * nq)
-    tensor_cores = dv == d and not values_in_keys and not flags and uses_tensor_cores(q.dtype, d)
+    tensor_cores = dv == d and not values_in_keys and not flags and sinks is None and uses_tensor_cores(q.dtype, d)
     base_rows = int(lib.lily_attention_prefill_mma_rows() if tensor_cores else lib.lily_attention_prefill_simt_rows())
     if tile_rows is not None and tile_rows != base_rows:
-        if not (tile_rows == int(lib.lily_attention_prefill_tc_rows()) and q.dtype == torch.bfloat16 and dv == d and not flags
+        if not (tile_rows == int(lib.lily_attention_prefill_tc_rows()) and q.dtype == torch.bfloat16 and dv == d and not flags and sinks is None
                 and lib.lily_attention_prefill_tc_takes(int(d), int(page_size))):
             raise KernelError(f"attention_prefill: no kernel with tiles of {tile_rows} rows for {q.dtype}, head size {d}, "
                               f"page size {page_size}")
@@ -714,7 +727,7 @@ def attention_prefill(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torc
     elif tensor_cores:
         _call("lily_attention_prefill_mma", *common, cap, keep_first, 0, 0, _stream())
     else:
-        _call("lily_attention_prefill_simt", *common, _dt(q), cap, -dv if values_in_keys else dv, keep_first, flags, 0, _stream())
+        _call("lily_attention_prefill_simt", *common, _dt(q), cap, -dv if values_in_keys else dv, keep_first, flags, 0, _p(sinks), _stream())
 
 
 _MERGED_SHIFTS = os.environ.get("LILY_B200_MERGED_SHIFTS", "1") != "0"
@@ -753,6 +766,11 @@ def all_values_sums(dtype: torch.dtype, tokens: int, nq: int, nkv: int, d: int, 
     return torch.empty((tokens, nq * nkv * dv), dtype=torch.float32, device=device)
 
 
+def _check_sinks(sinks: Optional[torch.Tensor], nq: int, other: bool) -> None:
+    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != nq or other):
+        raise KernelError("attention: a head's sinks are float32 [query heads] and come without the unit sink and all heads' values")
+
+
 def _attention_flags(sink: bool, all_values: bool, values_in_keys: bool, nkv: int, dv: int, out: torch.Tensor, rows: int) -> int:
     """The CUDA-core attention kernels' option bits: 1 the sink, 2 values of all kv heads, 4 float32 outputs."""
     if all_values:
@@ -777,12 +795,14 @@ def attention_decode(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch
                      out: torch.Tensor, scratch: Optional[torch.Tensor], splits: int, nq: int, nkv: int, d: int,
                      page_size: int, scale: float, window: Optional[int] = None, stages: int = 0,
                      softcap: Optional[float] = None, dv: Optional[int] = None, values_in_keys: bool = False,
-                     keep_first: int = 0, sink: bool = False, all_values: bool = False) -> None:
-    """``sink`` and ``all_values`` as in ``attention_prefill`` (CUDA-core kernel; the scratch then holds nkv * dv columns a head).
+                     keep_first: int = 0, sink: bool = False, all_values: bool = False,
+                     sinks: Optional[torch.Tensor] = None) -> None:
+    """``sink``, ``sinks`` and ``all_values`` as in ``attention_prefill`` (CUDA-core kernel; the scratch then holds nkv * dv columns a head).
     One query token per request (rows of ``q`` [requests, nq * d]) over ``seq_lens`` cached
     positions (the last ``window`` of them and the first ``keep_first``, where given), keys cut into ``splits`` ranges merged through ``scratch`` (float32).  ``stages`` (tensor-core
     kernel only): the key/value tiles a block holds, 0 for the default (``DecodePlan.stages``)."""
-    _dev(q, kv_layer, block_table, seq_lens, out, scratch)
+    _dev(q, kv_layer, block_table, seq_lens, out, scratch, sinks)
+    _check_sinks(sinks, nq, sink or all_values)
     requests = q.shape[0]
     planes = all_values and out.dim() == 3
     if q.dtype != kv_layer.dtype or out.dtype != (torch.float32 if all_values and not planes else q.dtype):
@@ -805,13 +825,13 @@ def attention_decode(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch
     if values_in_keys and latent_tcgen05(q.dtype, d, dv, page_size, nkv, softcap) and not stages:
         _call("lily_latent_attention_decode_tc", _p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"),
               block_table.shape[-1], _i32(seq_lens, "seq_lens"), _p(scratch), requests, splits, nq, d, dv, page_size,
-              int(window or 0), float(scale), kv_layer.shape[0], _stream())
+              int(window or 0), float(scale), kv_layer.shape[0], _p(sinks), _stream())
         if splits > 1:
             _call("lily_attention_combine", _p(scratch), _p(out), requests, nq, dv, splits, _dt(q), _stream())
     elif values_in_keys and latent_tensor_cores(q.dtype, d, dv, nkv, softcap) and not stages:
         _call("lily_latent_attention_decode_mma", _p(q), _p(kv_layer), _p(out), _i32(block_table, "block_table"),
               block_table.shape[-1], _i32(seq_lens, "seq_lens"), _p(scratch), requests, splits, nq, d, dv, page_size,
-              int(window or 0), float(scale), _stream())
+              int(window or 0), float(scale), _p(sinks), _stream())
         if splits > 1:
             _call("lily_attention_combine", _p(scratch), _p(out), requests, nq, dv, splits, _dt(q), _stream())
     elif on_tc:
@@ -823,7 +843,7 @@ def attention_decode(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch
             rows = requests * nkv if merged else requests
             if splits > 1 and (stages or rows * nkv * -(-(nq // nkv) // 16) > decode_clusters(d, splits, nq // nkv)):
                 launches["count"] += 1
-    elif dv == d and not values_in_keys and not flags and uses_tensor_cores(q.dtype, d):
+    elif dv == d and not values_in_keys and not flags and sinks is None and uses_tensor_cores(q.dtype, d):
         _call("lily_attention_decode_mma", *common, int(stages), cap, int(keep_first or 0) if window else 0, 0, 0, _stream())   # merges the splits itself (cluster, or combine behind)
         if splits > 1 and (stages or requests * nkv * -(-(nq // nkv) // 16) > decode_clusters(d, splits, nq // nkv)):
             launches["count"] += 1                                   # the combine kernel, launched inside
@@ -834,7 +854,7 @@ def attention_decode(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch
             _call("lily_attention_decode_simt", _p(q), _p(kv_layer), out[shift].data_ptr() if planes else _p(out),
                   _i32(block_table, "block_table"), block_table.shape[-1], _i32(seq_lens, "seq_lens"), _p(scratch), requests, splits,
                   nq, nkv, d, page_size, int(window or 0), float(scale), _dt(q), cap, -dv if values_in_keys else dv,
-                  int(keep_first or 0) if window else 0, (1 if sink else 0) if planes else flags, shift, _stream())
+                  int(keep_first or 0) if window else 0, (1 if sink else 0) if planes else flags, shift, _p(sinks), _stream())
             if splits > 1:
                 launches["count"] += 1          # the combine kernel, launched inside
 
@@ -984,14 +1004,16 @@ def attention_decode_fused(qkv: torch.Tensor, q_gain: Optional[torch.Tensor], k_
                            block_table: torch.Tensor, seq_lens: torch.Tensor, out: torch.Tensor,
                            scratch: Optional[torch.Tensor], splits: int, nq: int, nkv: int, d: int, rotary_dim: int,
                            page_size: int, scale: float, window: Optional[int] = None, write_kv: bool = True,
-                           stages: int = 0, softcap: Optional[float] = None) -> None:
+                           stages: int = 0, softcap: Optional[float] = None, row: Optional[int] = None) -> None:
     """``qk_norm_rope_write`` and ``attention_decode`` of a step in which every request brings one token, as one
     kernel: ``qkv`` is the projection's result ([requests, (nq + 2 nkv) d] in the cache's dtype, or float32 partial
     sums [splits, requests, ...]); the attention blocks finish their own query heads, and the block whose key range
-    holds the new position finishes the key and the value and writes them to the cache before it reads them."""
+    holds the new position finishes the key and the value and writes them to the cache before it reads them.
+    ``row`` as in ``qk_norm_rope_write``."""
     _dev(qkv, q_gain, k_gain, cos, sin, kv_layer, block_table, seq_lens, out, scratch)
     requests = qkv.shape[-2]
-    planes, stride = _summed(qkv, requests, (nq + 2 * nkv) * d, "attention_decode_fused qkv")
+    ld = int(row or (nq + 2 * nkv) * d)
+    planes, stride = _summed(qkv, requests, ld, "attention_decode_fused qkv")
     if not uses_tensor_cores(kv_layer.dtype, d) or out.dtype != kv_layer.dtype or qkv.dtype not in (kv_layer.dtype, torch.float32):
         raise KernelError(f"attention_decode_fused: cache {kv_layer.dtype}, qkv {qkv.dtype}, out {out.dtype}, head size {d}")
     if tuple(kv_layer.shape[1:]) != (2, nkv, page_size, d):
@@ -1007,7 +1029,7 @@ def attention_decode_fused(qkv: torch.Tensor, q_gain: Optional[torch.Tensor], k_
           _dt(q_gain) if q_gain is not None else _F32, float(eps), _p(cos), _p(sin), int(rotary_dim), int(write_kv),
           _p(kv_layer), _p(out), _i32(block_table, "block_table"), block_table.shape[-1], _i32(seq_lens, "seq_lens"),
           _p(scratch), requests, splits, nq, nkv, d, page_size, int(window or 0), float(scale), int(stages),
-          float(softcap or 0.0), _stream())
+          float(softcap or 0.0), ld, _stream())
     if splits > 1 and (stages or requests * nkv * -(-(nq // nkv) // 16) > decode_clusters(d, splits, nq // nkv)):
         launches["count"] += 1                                       # the combine kernel, launched inside
 
@@ -1028,6 +1050,17 @@ def sigmoid_gate(out: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
     n, cols = out.shape
     ptr, dt, splits, stride = _operand(gate, n, cols, "sigmoid_gate")
     _call("lily_sigmoid_gate", _p(out), _dt(out), ptr, dt, splits, stride, out.numel(), _stream())
+    return out
+
+
+def sigmoid_head_gate(out: torch.Tensor, gate: torch.Tensor, g0: int, heads: int) -> torch.Tensor:
+    """In place: head h's columns of ``out`` [tokens, heads * dv] times ``sigmoid(gate[t, g0 + h])``; ``gate`` [tokens, cols] in
+    either dtype, or float32 partial sums [splits, tokens, cols]."""
+    _dev(out, gate)
+    n, cols = out.shape
+    ld = gate.shape[-1]
+    ptr, dt, splits, stride = _operand(gate, n, ld, "sigmoid_head_gate")
+    _call("lily_sigmoid_head_gate", _p(out), _dt(out), ptr, dt, splits, stride, ld, int(g0), n, int(heads), cols // heads, _stream())
     return out
 
 
@@ -1413,25 +1446,25 @@ def group_rmsnorm_gate(y: torch.Tensor, gate: torch.Tensor, gain: torch.Tensor, 
 # ------------------------------------------------------------------------------ attention over a cached latent
 
 def latent_prepare(down: torch.Tensor, q0: int, q_rank: int, kv0: int, rank: int, rot: int, rotary_dim: int,
-                   q_gain: torch.Tensor, kv_gain: torch.Tensor, eps: float, cos: Optional[torch.Tensor],
+                   q_gain: Optional[torch.Tensor], kv_gain: torch.Tensor, eps: float, cos: Optional[torch.Tensor],
                    sin: Optional[torch.Tensor], positions: torch.Tensor, token_req: torch.Tensor,
-                   block_table: torch.Tensor, layer: torch.Tensor, page_size: int, write_kv: bool = True) -> torch.Tensor:
+                   block_table: torch.Tensor, layer: torch.Tensor, page_size: int, write_kv: bool = True) -> Optional[torch.Tensor]:
     """From a token's row of the stacked down-projection ``down`` (the cache's dtype, float32, or float32 partial sums
     [splits, tokens, cols]): the RMS-normed query
     latent (columns ``q0`` on, ``q_rank`` of them, gain ``q_gain``), returned as [tokens, q_rank] in the cache's
     dtype; and into the token's cache row [rank + rot] of ``layer`` [pages, page_size * (rank + rot)] the RMS-normed
     key/value latent (columns ``kv0`` on, gain ``kv_gain``) followed by the ``rot`` columns after it, the first
-    ``rotary_dim`` of them rotated in halves by the position's angles."""
+    ``rotary_dim`` of them rotated in halves by the position's angles.  ``q_rank`` 0: the queries have no latent (returns None)."""
     _dev(down, q_gain, kv_gain, cos, sin, positions, token_req, block_table, layer)
     tokens, cols = down.shape[-2:]
     ptr, dt, splits, stride = _operand(down, tokens, cols, "latent_prepare")
     if layer.dim() != 2 or layer.shape[1] != page_size * (rank + rot):
         raise KernelError(f"latent_prepare: cache layer {tuple(layer.shape)} does not hold pages of {page_size} rows of {rank + rot}")
-    if q_gain.dtype != torch.float32 or kv_gain.dtype != torch.float32:
+    if (q_rank and (q_gain is None or q_gain.dtype != torch.float32)) or kv_gain.dtype != torch.float32:
         raise KernelError("latent_prepare: gains are float32")
     if rotary_dim and (cos is None or cos.dtype != torch.float32 or cos.shape[-1] != rotary_dim // 2):
         raise KernelError("rotation tables must be float32 [positions, rotary_dim / 2]")
-    cq = torch.empty((tokens, q_rank), dtype=layer.dtype, device=down.device)
+    cq = torch.empty((tokens, q_rank), dtype=layer.dtype, device=down.device) if q_rank else None
     _call("lily_latent_prepare", ptr, dt, splits, stride, cols, q0, q_rank, kv0, rank, rot, rotary_dim, _p(q_gain),
           _p(kv_gain), float(eps), _p(cos), _p(sin), _i32(positions, "positions"), _i32(token_req, "token_req"),
           _i32(block_table, "block_table"), block_table.shape[-1], _p(layer), page_size, int(write_kv), _p(cq), tokens,
@@ -1488,14 +1521,15 @@ class ExpertRouting:
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, experts: int,
               scores: str = "softmax", renormalise: bool = True, shared_gate: bool = False,
-              outputs: Optional[int] = None) -> ExpertRouting:
+              outputs: Optional[int] = None, groups: int = 0, keep_groups: int = 0) -> ExpertRouting:
     """Scores of all router outputs (float32 logits ``router . h``, by this package's kernel for a float32 matrix; a matrix in
     ``h``'s bfloat16 takes a product with a float32 result, whose terms are exact; their softmax, or with ``scores`` "sigmoid" each one's
     sigmoid), the ``top`` largest scores (+ correction) chosen, their weights the scores themselves, over their sum with
     ``renormalise``; then the pairs of the first ``experts`` outputs (those with weights; the rest stand for the identity)
     grouped by expert.  ``shared_gate``: the matrix has one more row, the sigmoid of whose product is the token's gate for
     the shared expert.  ``outputs``: how many the router has where the matrix goes on behind its own rows (a bfloat16 matrix
-    whose rows are padded to a multiple of 8 gets the library's faster product)."""
+    whose rows are padded to a multiple of 8 gets the library's faster product).  ``groups`` equal runs of neighbouring outputs:
+    only those of the ``keep_groups`` runs with the largest sums of two choice scores can be chosen."""
     _dev(h, router, correction)
     tokens, width = h.shape
     if outputs is None:
@@ -1516,7 +1550,7 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.
         ints, [pairs, pairs, pairs, experts + 1, max_tiles, max_tiles, 1])
     weights = torch.empty((tokens, top), dtype=torch.float32, device=dev)
     gate = torch.empty((tokens,), dtype=torch.float32, device=dev) if shared_gate else None
-    how = (outputs, top, int(scores == "sigmoid"), int(renormalise), _p(chosen), _p(weights), _p(gate))
+    how = (outputs, top, int(scores == "sigmoid"), int(renormalise), int(groups), int(keep_groups), _p(chosen), _p(weights), _p(gate))
     if router.dtype == torch.bfloat16:
         z = linear_split(h, router)
         if z is None:
@@ -1540,7 +1574,7 @@ def grouped_library_takes(dtype: torch.dtype, width: int, ff: int) -> bool:
             and not _OWN_GROUPED)
 
 
-EXPERT_ACTIVATIONS = {"swish_clamped": 0, "silu": 1}
+EXPERT_ACTIVATIONS = {"swish_clamped": 0, "silu": 1, "relu2": 2}      # "relu2": ungated
 
 
 def moe_experts(h: torch.Tensor, routing: ExpertRouting, w_gate_up: torch.Tensor, w_down: torch.Tensor, limit: float = 0.0,
@@ -1550,8 +1584,10 @@ def moe_experts(h: torch.Tensor, routing: ExpertRouting, w_gate_up: torch.Tensor
     width] (an expert's gate rows, then its up rows), ``w_down`` [experts, width, ff].  An expert computes
     ``W_down (g sigmoid(alpha g) (u + 1))`` with ``g = min(W_gate h, limit)``, ``u = clamp(W_up h, -limit, limit)``, or, with
     ``activation`` "silu", ``W_down (silu(W_gate h) (W_up h))``; a choice beyond the experts that have weights contributes
-    ``h`` itself.  ``weight_on_input``: a pair's weight multiplies what its expert is given instead of what it gives.
+    ``h`` itself.  ``activation`` "relu2": ungated experts, ``W_down max(W_up h, 0)^2``, with ``w_gate_up`` [experts, ff, width] the
+    up rows alone.  ``weight_on_input``: a pair's weight multiplies what its expert is given instead of what it gives.
     ``shared``: the shared expert's output ([tokens, width], or float32 partial sums), added times ``routing.gate``."""
+    gated = activation != "relu2"
     if activation not in EXPERT_ACTIVATIONS:
         raise KernelError(f"moe_experts: no activation {activation!r}; have {sorted(EXPERT_ACTIVATIONS)}")
     _dev(h, w_gate_up, w_down, shared)
@@ -1570,16 +1606,19 @@ def moe_experts(h: torch.Tensor, routing: ExpertRouting, w_gate_up: torch.Tensor
         _call("lily_moe_gather", _p(h), width, _p(r.offsets), experts, _p(r.order), r.top, pairs, _p(rows), _stream())
         gate_up = torch._grouped_mm(rows, w_gate_up.transpose(1, 2), offs=ends)
         act = torch.empty((pairs, ff), dtype=h.dtype, device=h.device)
-        _call("lily_moe_activation", _p(gate_up), ff, pairs, _p(act), act_code, float(limit), float(alpha), in_weight, _p(r.offsets),
-              experts, _p(r.order), _stream())
+        if not gated:
+            _call("lily_moe_relu2", _p(gate_up), ff, pairs, _p(act), in_weight, _p(r.offsets), experts, _p(r.order), _stream())
+        else:
+            _call("lily_moe_activation", _p(gate_up), ff, pairs, _p(act), act_code, float(limit), float(alpha), in_weight,
+                  _p(r.offsets), experts, _p(r.order), _stream())
         y = torch._grouped_mm(act, w_down.transpose(1, 2), offs=ends)
     else:
         y = torch.empty((max(pairs, 1), width), dtype=torch.float32, device=h.device)
         if experts:
-            if w_gate_up.dtype != h.dtype or w_down.dtype != h.dtype or tuple(w_gate_up.shape) != (experts, 2 * ff, width):
+            if w_gate_up.dtype != h.dtype or w_down.dtype != h.dtype or tuple(w_gate_up.shape) != (experts, 2 * ff if gated else ff, width):
                 raise KernelError(f"moe_experts: weights {tuple(w_gate_up.shape)} / {tuple(w_down.shape)} {w_down.dtype} for inputs {tuple(h.shape)} {h.dtype}")
             act = torch.empty((max(pairs, 1), ff), dtype=h.dtype, device=h.device)
-            _call("lily_moe_gemm", 0, _p(h), h.stride(0), _p(w_gate_up), ff, width, _p(r.offsets), _p(r.order), r.top,
+            _call("lily_moe_gemm", 0 if gated else 2, _p(h), h.stride(0), _p(w_gate_up), ff, width, _p(r.offsets), _p(r.order), r.top,
                   _p(r.tile_expert), _p(r.tile_row), _p(r.tile_count), r.max_tiles, _p(act), act_code, float(limit), float(alpha),
                   in_weight, _dt(h), _stream())
             _call("lily_moe_gemm", 1, _p(act), ff, _p(w_down), width, ff, _p(r.offsets), _p(r.order), r.top, _p(r.tile_expert),
@@ -1708,6 +1747,32 @@ def add_normed(resid: torch.Tensor, delta: torch.Tensor, post_gain: torch.Tensor
     _call("lily_add_normed_rmsnorm", _p(resid), ptr, dt, splits, stride, _p(post_gain), float(post_eps), float(mult), None, _F32, _p(out),
           _dt(out) if out is not None else _F32, None, n, width, 0.0, 1, int(bool(normalise)), _stream())
     return resid if out is None else out
+
+
+def add_tanh_norm(resid: torch.Tensor, delta: Optional[torch.Tensor], post, mult: float, pre, out_dtype: Optional[torch.dtype],
+                  rows: Optional[torch.Tensor] = None, write_residual: bool = True) -> Optional[torch.Tensor]:
+    """``resid += mult * (gain tanh(alpha delta) + shift)`` with ``post`` = (alpha, gain, shift), or ``resid += mult * delta``
+    without; then the new rows as ``gain tanh(alpha v) + shift`` with ``pre``'s numbers (the rows themselves without ``pre``) in
+    ``out_dtype`` (None: the add alone).  ``delta`` [tokens, width] in either dtype, float32 partial sums [splits, tokens,
+    width], or None; gains and shifts float32 [width].  With ``rows`` only those tokens' outputs are formed and the stream is
+    left as it is."""
+    n, width = resid.shape
+    for p in (post, pre):
+        if p is not None and (p[1].dtype != torch.float32 or p[1].numel() != width or p[2].dtype != torch.float32 or p[2].numel() != width):
+            raise KernelError("add_tanh_norm: gains and shifts are float32 vectors of the row's length")
+    _dev(resid, delta, rows, *(post or ())[1:], *(pre or ())[1:])
+    if resid.dtype != torch.float32:
+        raise KernelError("the residual stream is float32")
+    ptr, dt, splits, stride = _operand(delta, n, width, "add_tanh_norm delta") if delta is not None else (None, _F32, 1, 0)
+    n_out = n if rows is None else rows.numel()
+    out = None if out_dtype is None else torch.empty((n_out, width), dtype=out_dtype, device=resid.device)
+    if out is None and (rows is not None or delta is None):
+        return None
+    a, g, s = post or (0.0, None, None)
+    b, w, c = pre or (0.0, None, None)
+    _call("lily_add_tanh_norm", _p(resid), ptr, dt, splits, stride, float(a), _p(g), _p(s), float(mult), float(b), _p(w), _p(c), _p(out),
+          _dt(out) if out is not None else _F32, _i32(rows, "rows"), n_out, width, int(bool(write_residual and rows is None)), _stream())
+    return out
 
 
 def activation(x: torch.Tensor, out_dtype: torch.dtype, activation: str = "relu2",
@@ -1873,4 +1938,53 @@ def selective_scan(x: torch.Tensor, low: torch.Tensor, b_col: int, step: torch.T
     if plan.num_direct:
         _call("lily_selective_scan", *common, plan.num_direct, tokens, inner, n, _dt(x), _i32(plan.direct, "direct"), None, None,
               0, None, None, _stream())
+    return out
+
+
+# ------------------------------------------------------------------------------ matrix memory with exponential gates
+
+def mlstm_max_head_dim() -> int:
+    return int(library().lily_mlstm_max_head_dim())
+
+
+def mlstm_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, gates: torch.Tensor, i_col: int, f_col: int, i_bias: torch.Tensor,
+               f_bias: torch.Tensor, cap: float, q_scale: float, state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor,
+               requests: int, heads: int, d: int, dv: int) -> Tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+    """The recurrence of the matrix memory over each request's new tokens, from and to ``state[slot]`` (float32, [heads, dv + 1,
+    d] with the normaliser as the last column, then the heads' scales, which ``mlstm_out`` writes).  ``proj`` [tokens, width]
+    holds q and k (heads x d) and v (heads x dv) from their columns on, ``gates`` [tokens, width] the gates' inputs before their
+    biases (either may be float32 partial sums).  q is multiplied by ``q_scale``.  Returns float32 (S^T q [tokens, heads * dv],
+    n . q [tokens, heads], m [tokens, heads])."""
+    _dev(proj, gates, i_bias, f_bias, state, cu_seqlens, slots)
+    n, ld = proj.shape[-2:]
+    gn, gld = gates.shape[-2:]
+    if gn != n or max(q_col + heads * d, k_col + heads * d, v_col + heads * dv) > ld or max(i_col, f_col) + heads > gld:
+        raise KernelError("mlstm_scan: columns out of range")
+    if i_bias.dtype != torch.float32 or f_bias.dtype != torch.float32 or i_bias.numel() != heads or f_bias.numel() != heads \
+            or state.dtype != torch.float32 or state.dim() != 2:
+        raise KernelError("mlstm_scan: biases [heads] and state are float32")
+    y = torch.empty((n, heads * dv), dtype=torch.float32, device=proj.device)
+    nm = torch.empty((2, n, heads), dtype=torch.float32, device=proj.device)
+    _call("lily_mlstm_scan", *_operand(proj, n, ld, "mlstm_scan"), ld, int(q_col), int(k_col), int(v_col),
+          *_operand(gates, n, gld, "mlstm_scan gates"), gld, int(i_col), int(f_col), _p(i_bias), _p(f_bias), float(cap), float(q_scale),
+          _p(state), state.stride(0), _p(y), nm[0].data_ptr(), nm[1].data_ptr(), _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots"), None,
+          int(requests), heads, d, dv, _stream())
+    return y, nm[0], nm[1]
+
+
+def mlstm_out(y: torch.Tensor, nq: torch.Tensor, m: torch.Tensor, gate: torch.Tensor, gate_col: int, gain: torch.Tensor, floor: float,
+              eps: float, state: torch.Tensor, m_off: int, cu_seqlens: torch.Tensor, token_req: torch.Tensor, slots: torch.Tensor,
+              out_dtype: torch.dtype) -> torch.Tensor:
+    """``o = y / (max(|nq|, exp(-m)) + floor)`` per head, divided by its root mean square, times ``gain`` (float32 [heads * dv]),
+    times ``sigmoid(gate[:, gate_col:])``; the last token's m of each request goes to ``state[slot, m_off:]``."""
+    _dev(y, nq, m, gate, gain, state, cu_seqlens, token_req, slots)
+    tokens, heads = nq.shape
+    ld = gate.shape[-1]
+    inner = y.shape[1]
+    if gain.dtype != torch.float32 or gain.numel() != inner or gate_col + inner > ld:
+        raise KernelError("mlstm_out: float32 gain [heads * dv], gate columns inside the row")
+    out = torch.empty((tokens, inner), dtype=out_dtype, device=y.device)
+    _call("lily_mlstm_out", _p(y), _p(nq), _p(m), *_operand(gate, tokens, ld, "mlstm_out"), ld, int(gate_col), _p(gain), float(floor), float(eps),
+          _p(out), _dt(out), _p(state), state.stride(0), int(m_off), _i32(cu_seqlens, "cu_seqlens"), _i32(token_req, "token_req"),
+          _i32(slots, "slots"), tokens, heads, inner // heads, _stream())
     return out

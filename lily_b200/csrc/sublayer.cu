@@ -7,6 +7,9 @@
 //                        out = v / sqrt(mean(v^2) + eps) * weight                        (the norm ahead of the next one; or,
 //                                                                                         without `weight`, out = v: a sublayer
 //                                                                                         that reads the stream itself)
+//   add_tanh_norm:       v = resid + mult * (gain_post * tanh(alpha_post * delta) + shift_post)      (or v = resid + mult * delta)
+//                        out = gain * tanh(alpha * v) + shift                            (norms without a mean or a variance: no sum
+//                                                                                         over the row, every column by itself)
 //   activation:          out = act(in), act = SiLU, the tanh form of GELU, the square of max(., 0), or xIELU
 //
 // `delta` and `in` may be the activation dtype, float32, or the float32 partial sums of a split-k product.  Sums of
@@ -217,6 +220,78 @@ __global__ void add_normed_rmsnorm_cluster_kernel(const NormedAddArgs a) {
     dst[3] = from_float<T>((v.w * inv) * gain_at(a.weight, a.weight_bf16, i + 3));
 }
 
+struct TanhNorm {
+    float alpha;
+    const float* gain;        // [hidden]; null: no such norm
+    const float* shift;       // [hidden]
+};
+
+struct TanhAddArgs {
+    float* resid;             // [tokens, hidden]
+    Operand delta;            // [tokens, hidden]; a null pointer: nothing is added
+    TanhNorm post, pre;
+    void* out;                // [rows or tokens, hidden]; null: the add alone
+    const int* rows;          // null: every token; else the tokens whose output is wanted (nothing is written back then)
+    int hidden, n_out;
+    float mult;
+    int write_residual;
+};
+
+// grid (ceil(hidden / (VEC * blockDim)), ceil(rows / ROWS)): a thread owns VEC neighbouring columns of ROWS rows, so that gains
+// and shifts read once serve several rows.
+template <typename T, int VEC, int ROWS>
+__global__ void add_tanh_norm_kernel(const TanhAddArgs a) {
+    pdl_enter_small();
+    const int i = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (i >= a.hidden) return;
+    float pg[VEC], ps[VEC], g[VEC], s[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+        pg[e] = a.post.gain ? a.post.gain[i + e] : 1.f;
+        ps[e] = a.post.gain ? a.post.shift[i + e] : 0.f;
+        g[e] = a.pre.gain ? a.pre.gain[i + e] : 1.f;
+        s[e] = a.pre.gain ? a.pre.shift[i + e] : 0.f;
+    }
+    float v[ROWS][VEC], d[ROWS][VEC];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const int m = blockIdx.y * ROWS + r;
+        if (m >= a.n_out) break;
+        const size_t src = (size_t)(a.rows ? a.rows[m] : m) * a.hidden + i;
+        if (VEC == 4) {
+            *reinterpret_cast<float4*>(v[r]) = *reinterpret_cast<const float4*>(a.resid + src);
+            *reinterpret_cast<float4*>(d[r]) = a.delta.p ? a.delta.four(src) : make_float4(0.f, 0.f, 0.f, 0.f);
+        } else {
+            v[r][0] = a.resid[src];
+            d[r][0] = a.delta.p ? a.delta(src) : 0.f;
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const int m = blockIdx.y * ROWS + r;
+        if (m >= a.n_out) break;
+        if (a.delta.p) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                const float u = a.post.gain ? fmaf(tanhf(a.post.alpha * d[r][e]), pg[e], ps[e]) : d[r][e];
+                v[r][e] = fmaf(a.mult, u, v[r][e]);
+            }
+            if (a.write_residual) {
+                float* dst = a.resid + (size_t)(a.rows ? a.rows[m] : m) * a.hidden + i;
+                if (VEC == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(v[r]);
+                else dst[0] = v[r][0];
+            }
+        }
+        if (a.out == nullptr) continue;
+        T* dst = (T*)a.out + (size_t)m * a.hidden + i;
+        float o[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) o[e] = a.pre.gain ? fmaf(tanhf(a.pre.alpha * v[r][e]), g[e], s[e]) : v[r][e];
+        if constexpr (VEC == 4) store_four<T>(dst, make_float4(o[0], o[1], o[2], o[3]));
+        else dst[0] = from_float<T>(o[0]);
+    }
+}
+
 // act: 0 SiLU, 1 the tanh form of GELU, 2 the square of max(., 0), 3 xIELU with its two factors
 __device__ __forceinline__ float activate(int act, float z, float p0, float p1) {
     if (act == 3) return xielu(z, p0, p1);
@@ -333,6 +408,36 @@ LILY_API int lily_add_normed_rmsnorm(float* resid, const void* delta, int delta_
     else { if (vec) GO(float, 4); else GO(float, 1); }
 #undef GO
     LILY_CHECK_LAUNCH("add_normed_rmsnorm");
+    return 0;
+}
+
+// post_gain / pre_gain null: no such norm; delta null: nothing is added; out null: the add alone.
+LILY_API int lily_add_tanh_norm(float* resid, const void* delta, int delta_dtype, int delta_splits, size_t delta_stride, float post_alpha,
+                                const float* post_gain, const float* post_shift, float mult, float alpha, const float* gain, const float* shift,
+                                void* out, int out_dtype, const int* rows, int n_out, int hidden, int write_residual, cudaStream_t stream) {
+    if (n_out == 0) return 0;
+    LILY_REQUIRE(hidden > 0, "add_tanh_norm: width %d", hidden);
+    LILY_REQUIRE(delta_splits >= 1 && (delta_splits == 1 || delta_dtype == kF32), "add_tanh_norm: only float32 partial sums come in several splits");
+    LILY_REQUIRE((post_gain == nullptr) == (post_shift == nullptr) && (gain == nullptr) == (shift == nullptr), "add_tanh_norm: gains and shifts come together");
+    LILY_REQUIRE(!(rows && write_residual), "add_tanh_norm: gathered rows are not written back");
+    TanhAddArgs a{};
+    a.resid = resid; a.delta = Operand{delta, delta_dtype == kBF16, delta_splits, delta_stride};
+    a.post = TanhNorm{post_alpha, post_gain, post_shift}; a.pre = TanhNorm{alpha, gain, shift};
+    a.out = out; a.rows = rows; a.hidden = hidden; a.n_out = n_out; a.mult = mult; a.write_residual = write_residual;
+    const bool vec = hidden % 4 == 0 && a.delta.vector_ok() && ((uintptr_t)resid & 15) == 0 && ((uintptr_t)out & 15) == 0;
+    const int cols = vec ? hidden / 4 : hidden, threads = cols >= 128 ? 128 : (cols + 31) / 32 * 32;
+    const int per = vec && n_out >= 1024 ? 4 : 1;
+    dim3 grid((cols + threads - 1) / threads, (n_out + per - 1) / per);
+    LILY_REQUIRE(grid.y <= 65535, "add_tanh_norm: %d rows", n_out);
+#define GO(T)                                                                                                       \
+    do {                                                                                                            \
+        if (per == 4) launch_pdl(add_tanh_norm_kernel<T, 4, 4>, grid, dim3(threads), 0, stream, a);                 \
+        else if (vec) launch_pdl(add_tanh_norm_kernel<T, 4, 1>, grid, dim3(threads), 0, stream, a);                 \
+        else launch_pdl(add_tanh_norm_kernel<T, 1, 1>, grid, dim3(threads), 0, stream, a);                          \
+    } while (0)
+    if (out_dtype == kBF16) GO(__nv_bfloat16); else GO(float);
+#undef GO
+    LILY_CHECK_LAUNCH("add_tanh_norm");
     return 0;
 }
 

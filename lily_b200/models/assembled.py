@@ -3,7 +3,7 @@
 The schedule is walked as data.  For each position of the schedule, every mixer of its block that
 asks for paged keys and values gets a layer of its own in the cache group that matches the need
 (or, with ``reads``, borrows the layer of the same mixer at an earlier position and writes
-nothing); every mixer that asks for per-request state gets a state tensor of its own.  The same
+nothing; a layer that is lent keeps its keys as long as the furthest-looking of its readers needs them); every mixer that asks for per-request state gets a state tensor of its own.  The same
 block may therefore run twice with separate caches.  The embedding may be scaled and the logits
 scaled and soft-capped (``ModelSpec.embed_scale``, ``logit_scale``, ``logit_softcap``).
 
@@ -14,6 +14,7 @@ before the final norm, as lily/models/llama.py:199-205 gathers the last row of e
 
 from __future__ import annotations
 
+import dataclasses
 from typing import Dict, List, Optional, Tuple
 
 import torch
@@ -45,6 +46,7 @@ class AssembledModel:
         self.entry_state: List[List[Optional[int]]] = []
         group_of: Dict[CacheNeed, int] = {}
         counts: List[int] = []
+        kept = self._kept_keys(spec)
         for pos, entry in enumerate(spec.schedule):
             if not (0 <= entry.block < len(self.blocks)):
                 raise ValueError(f"schedule position {pos} names block {entry.block} of {len(self.blocks)}")
@@ -67,12 +69,9 @@ class AssembledModel:
                     other = owners[k].cache_need()
                     if (other.kv_heads, other.head_dim, other.v_head_dim) != (need.kv_heads, need.head_dim, need.v_head_dim):
                         raise ValueError(f"schedule position {pos} cannot read a cache of another shape")
-                    if other.window is not None and (need.window is None or need.window > other.window):
-                        # the owner's group gives pages back once its window has passed them
-                        raise ValueError(f"schedule position {pos} looks back {need.window or 'over all'} keys but reads "
-                                         f"a cache that keeps the last {other.window}")
                     caches.append((lent[0], lent[1], False))
                 else:
+                    need = dataclasses.replace(need, window=kept[pos, k][0], keep_first=kept[pos, k][1])
                     if need not in group_of:
                         group_of[need] = len(counts)
                         counts.append(0)
@@ -88,6 +87,23 @@ class AssembledModel:
             self.entry_cache.append(caches)
             self.entry_state.append(states)
         self.cache_groups = [(need, counts[g]) for need, g in sorted(group_of.items(), key=lambda kv: kv[1])]
+
+    def _kept_keys(self, spec: ModelSpec) -> Dict[Tuple[int, int], Tuple[Optional[int], int]]:
+        """(window, first positions) that the pages of each cache-owning (position, mixer) have to keep: its own, or those of
+        a reader that looks further back (a group gives pages back once its window has passed them)."""
+        kept: Dict[Tuple[int, int], Tuple[Optional[int], int]] = {}
+        for pos, entry in enumerate(spec.schedule):
+            owner = pos
+            while spec.schedule[owner].reads is not None and 0 <= spec.schedule[owner].reads < owner:
+                owner = spec.schedule[owner].reads
+            for k, mixer in enumerate(self.blocks[entry.block].mixers if 0 <= entry.block < len(self.blocks) else ()):
+                need = mixer.cache_need()
+                if need is None:
+                    continue
+                window, first = kept.get((owner, k), (need.window, need.keep_first))
+                window = None if window is None or need.window is None else max(window, need.window)
+                kept[owner, k] = (window, max(first, need.keep_first) if window is not None else 0)
+        return kept
 
     @property
     def graph_safe(self) -> bool:

@@ -6,7 +6,10 @@ leaves q in a buffer and writes k and v into the token's page; attention runs ov
 (split-key decode kernel for requests that bring one token, prefill kernel for portions); the
 output projection closes the part.  Options of the spec: a value head size of its own (``v_head_dim``), scores soft-capped
 to ``softcap * tanh(score / softcap)``, an output gate (the concatenated heads times ``sigmoid(W_g x)`` ahead of the
-output projection, W_g reading the mixer's input), rotation of interleaved pairs (the rows of the q and k projections
+output projection, W_g reading the mixer's input; or one gate a head, ``head_gate``, whose rows then ride in the stacked
+matrix), keys and values of another run's cache (``own_kv`` False), q and k heads brought to unit root mean square without a
+gain (``qk_gain`` False; a rotation leaves a head's root mean square as it is, so it does not matter which of the two comes
+first), rotation of interleaved pairs (the rows of the q and k projections
 are reordered once at load time, see ``rope.pairing_order``), and the checkpoint's own tensor names.  How a step's attention is cut (key ranges, kernel forms, tile
 lists) is this part's own plan, made once a step from the batch's host fields by asking the kernels
 (``ops.plan_decode_attention``, ``ops.prefill_tile_rows``, ``ops.prefill_tiles``); the step function
@@ -58,6 +61,9 @@ class AttentionSpec:
     # (1 - lambda) v + lambda v_first with lambda the scalar tensor of role "v_blend" and v_first the kept values of
     # the same token; layers that share have one kv_heads x v_head_dim
     v_share: Optional[str] = None
+    qk_gain: bool = True                  # with ``qk_norm``: the checkpoint holds gains; False: the heads are divided alone
+    head_gate: bool = False               # head h's output times sigmoid(W_g x)_h, one number a head
+    own_kv: bool = True                   # False: keys and values are another run's (as cached); this mixer projects none
 
     @property
     def value_dim(self) -> int:
@@ -77,6 +83,8 @@ class AttentionSpec:
     @property
     def projected(self) -> int:
         """Columns of the stacked q, k and v projections."""
+        if not self.own_kv:
+            return self.num_heads * self.head_dim
         return (self.num_heads + self.num_kv_heads) * self.head_dim + self.num_kv_heads * self.value_dim
 
 
@@ -118,6 +126,11 @@ class Attention(Mixer):
         self.v_blend = None
         if spec.keep_first and not spec.window:
             raise ValueError("first positions are kept in sight only beside a window")
+        if (spec.head_gate or not spec.own_kv) and (spec.bias or spec.conv_taps or spec.v_norm or spec.v_share):
+            raise ValueError("a gate a head, and another run's keys and values, come without biases, convolution, normed or shared values")
+        if spec.head_gate and spec.out_gate:
+            raise ValueError("the output gate is one number a column or one a head")
+        self.row = None                       # columns of the product where its rows go on behind the heads
         if spec.conv_taps < 0 or (spec.conv_taps and spec.bias):
             raise ValueError("the short convolution has at least one tap and comes without biases")
         self.conv_w = None
@@ -140,9 +153,12 @@ class Attention(Mixer):
         q, kv = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim
         heads_out = s.num_heads * s.value_dim
         out = {f"{p}.{s.name('q')}": TensorSpec((q, s.hidden_size)),
-               f"{p}.{s.name('k')}": TensorSpec((kv, s.hidden_size)),
-               f"{p}.{s.name('v')}": TensorSpec((s.num_kv_heads * s.value_dim, s.hidden_size)),
                f"{p}.{s.name('o')}": TensorSpec((s.hidden_size, heads_out))}
+        if s.own_kv:
+            out.update({f"{p}.{s.name('k')}": TensorSpec((kv, s.hidden_size)),
+                        f"{p}.{s.name('v')}": TensorSpec((s.num_kv_heads * s.value_dim, s.hidden_size))})
+        if s.head_gate:
+            out[f"{p}.{s.name('g')}"] = TensorSpec((s.num_heads, s.hidden_size))
         if s.out_gate:
             out[f"{p}.{s.name('g')}"] = TensorSpec((heads_out, s.hidden_size))
         if s.conv_taps:
@@ -155,7 +171,7 @@ class Attention(Mixer):
                         f"{p}.{s.name('v_bias')}": TensorSpec((s.num_kv_heads * s.value_dim,), role="matrix")})
             if s.out_bias:
                 out[f"{p}.{s.name('o_bias')}"] = TensorSpec((s.hidden_size,), role="matrix")
-        if s.qk_norm:
+        if s.qk_norm and s.qk_gain:
             out.update({f"{p}.{s.name('q_norm')}": TensorSpec((s.head_dim,), role="vector", init="gain"),
                         f"{p}.{s.name('k_norm')}": TensorSpec((s.head_dim,), role="vector", init="gain")})
         if s.talk:
@@ -167,18 +183,29 @@ class Attention(Mixer):
     def load(self, get) -> None:
         s, p = self.spec, self.prefix
         q, kv = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim
-        wq, wk = get(f"{p}.{s.name('q')}"), get(f"{p}.{s.name('k')}")
+        wq = get(f"{p}.{s.name('q')}")
+        wk = get(f"{p}.{s.name('k')}") if s.own_kv else None
         if self.position is not None and getattr(self.position, "interleaved", False):
             # pairs (2i, 2i + 1) become (i, i + rotary_dim / 2) in every q and k head alike: the scores are the same
             from lily_b200.parts.rope import pairing_order
             order = pairing_order(s.head_dim, self.position.rotary_dim).to(wq.device)
             wq = wq.view(s.num_heads, s.head_dim, -1)[:, order].reshape(q, -1)
-            wk = wk.view(s.num_kv_heads, s.head_dim, -1)[:, order].reshape(kv, -1)
-        self.w_qkv = torch.empty((q + kv + s.num_kv_heads * s.value_dim, s.hidden_size), dtype=wq.dtype, device=wq.device)
+            if wk is not None:
+                wk = wk.view(s.num_kv_heads, s.head_dim, -1)[:, order].reshape(kv, -1)
+        rows = s.projected + (s.num_heads if s.head_gate else 0)
+        if s.head_gate:
+            rows += -rows % 8                                              # zero rows: the product's rows stay whole 16-byte pieces
+        self.w_qkv = torch.empty((rows, s.hidden_size), dtype=wq.dtype, device=wq.device)
         self.w_qkv[:q].copy_(wq)
-        self.w_qkv[q:q + kv].copy_(wk)
+        if wk is not None:
+            self.w_qkv[q:q + kv].copy_(wk)
         del wq, wk
-        self.w_qkv[q + kv:].copy_(get(f"{p}.{s.name('v')}"))
+        if s.own_kv:
+            self.w_qkv[q + kv:s.projected].copy_(get(f"{p}.{s.name('v')}"))
+        if s.head_gate:
+            self.w_qkv[s.projected:s.projected + s.num_heads].copy_(get(f"{p}.{s.name('g')}"))
+            self.w_qkv[s.projected + s.num_heads:].zero_()
+        self.row = rows if s.head_gate or not s.own_kv else None
         self.w_o = get(f"{p}.{s.name('o')}").contiguous()
         if s.out_gate:
             self.w_g = get(f"{p}.{s.name('g')}").contiguous()
@@ -197,7 +224,9 @@ class Attention(Mixer):
         if s.v_share:
             blend = get(f"{p}.{s.name('v_blend')}")                              # the first layer's is loaded and not used
             self.v_blend = float(blend.float().item()) if s.v_share == "blend" else None
-        if s.qk_norm:
+        if s.qk_norm and not s.qk_gain:
+            self.q_gain = self.k_gain = torch.ones((s.head_dim,), dtype=torch.float32, device=self.w_qkv.device)
+        elif s.qk_norm:
             self.q_gain = get(f"{p}.{s.name('q_norm')}")
             self.k_gain = get(f"{p}.{s.name('k_norm')}")
             if self.q_gain.dtype != self.k_gain.dtype:
@@ -210,7 +239,7 @@ class Attention(Mixer):
         shared by every layer with the same sizes (``batch.plan``)."""
         s, ops = self.spec, self.ctx.ops
         key = ("attention", group, s.num_heads, s.num_kv_heads, s.head_dim, dtype, page, s.value_dim, bool(s.softcap),
-               bool(s.keep_first), bool(s.conv_taps), s.sink, s.talk)
+               bool(s.keep_first), bool(s.conv_taps), s.sink, s.talk, s.window)
         sized = {} if s.value_dim == s.head_dim else {"dv": s.value_dim}      # options go to the kernels' faces only
         capped = {"softcap": s.softcap} if s.softcap else {}                  # where the spec sets them
         if s.keep_first:
@@ -230,9 +259,10 @@ class Attention(Mixer):
             nd = b.num_decode
             # the rows the decode kernel sees (with mixed heads it may run every kv head's values in one launch)
             seen = ops.all_values_decode_rows(dtype, nd, s.num_kv_heads, s.head_dim, s.value_dim) if s.talk else nd
-            decode = ops.plan_decode_attention(dtype, seen, s.num_heads, s.num_kv_heads, s.head_dim, b.max_decode_len,
+            keys = min(b.max_decode_len, s.window + int(s.keep_first)) if s.window else b.max_decode_len      # of one row
+            decode = ops.plan_decode_attention(dtype, seen, s.num_heads, s.num_kv_heads, s.head_dim, keys,
                                                even=b.decode_even, **sized)
-            if decode != ops.plan_decode_attention(dtype, seen, s.num_heads, s.num_kv_heads, s.head_dim, b.max_decode_len,
+            if decode != ops.plan_decode_attention(dtype, seen, s.num_heads, s.num_kv_heads, s.head_dim, keys,
                                                    even=not b.decode_even, **sized):
                 b.even_asked = True              # a captured step with this plan serves batches of this kind only
             if (s.conv_taps or s.v_norm or s.v_share) and decode.fused:
@@ -255,6 +285,8 @@ class Attention(Mixer):
         if s.sink or s.talk:
             kept = dict(kept, sink=s.sink, all_values=s.talk)
         table = batch.block_tables[cache.group]
+        longer = {} if self.row is None else {"row": self.row}
+        write_cache = write_cache and s.own_kv
         plan = self._plan(batch, cache.group, cache.data.dtype, page)
         if s.conv_taps:
             chunk = ops.SSM_CHUNK
@@ -274,9 +306,11 @@ class Attention(Mixer):
             out = torch.empty((nd, s.num_heads * s.head_dim), dtype=cache.data.dtype, device=cache.data.device)
             ops.attention_decode_fused(qkv, self.q_gain, self.k_gain, s.norm_eps, cos, sin, cache.data, table, batch.seq_lens,
                                        out, scratch, dec.splits, s.num_heads, s.num_kv_heads, s.head_dim, rotary_dim, page,
-                                       self.scale, s.window, write_kv=write_cache, stages=dec.stages, **capped)
+                                       self.scale, s.window, write_kv=write_cache, stages=dec.stages, **capped, **longer)
             if gate is not None:
                 ops.sigmoid_gate(out, gate)
+            if s.head_gate:
+                ops.sigmoid_head_gate(out, qkv, s.projected, s.num_heads)
             return ops.linear_auto(out, self.w_o, self.b_o)
         values = {}
         if s.v_norm or s.v_share:
@@ -290,7 +324,7 @@ class Attention(Mixer):
                     values["v_blend"] = self.v_blend
         q = ops.qk_norm_rope_write(qkv, self.q_gain, self.k_gain, s.norm_eps, cos, sin, batch.positions,
                                    batch.token_req, table, cache.data, s.num_heads, s.num_kv_heads, s.head_dim,
-                                   rotary_dim, page, write_kv=write_cache, **sized, **values)
+                                   rotary_dim, page, write_kv=write_cache, **sized, **values, **longer)
         if s.talk:
             out = ops.all_values_sums(q.dtype, q.shape[0], s.num_heads, s.num_kv_heads, s.head_dim, dv, q.device)
         else:
@@ -308,6 +342,8 @@ class Attention(Mixer):
                                   tile_rows=plan.tile_rows, **capped, **sized, **kept)
         if gate is not None:
             ops.sigmoid_gate(out, gate)
+        if s.head_gate:
+            ops.sigmoid_head_gate(out, qkv, s.projected, s.num_heads)
         if s.talk:
             out = ops.head_mix(out, self.talk, s.num_heads, s.num_kv_heads, dv, q.dtype)
         return ops.linear_auto(out, self.w_o, self.b_o)

@@ -27,6 +27,7 @@ Interfaces
                         ``graph_safe``) and may keep a plan of its own there (``batch.plan``).
 ``FeedForward.forward(x, batch)`` -> [tokens, hidden] delta.
 ``Norm.forward(residual, delta, delta_bias, rows, write_residual)`` -> normed activations.
+``Norm.behind(mult)``   -> for a norm behind a sublayer: what turns the sublayer's output into a pending delta.
 ``Block.mixers``     -> the mixers of the block, in a fixed order; each run of the block gets a
                         cache layer and a state tensor for each of them (``RunSlots``).
 ``Block.forward(residual, delta, batch, run)`` -> next pending delta (a tensor, or a tuple of tensors to be summed).
@@ -203,7 +204,7 @@ def _load_builtin_parts() -> None:
     global _BUILTINS
     if not _BUILTINS:
         _BUILTINS = True
-        from lily_b200.parts import (attention, block, delta_rule, diff_attention, experts, latent_attention, mlp, norm, rope,  # noqa: F401
+        from lily_b200.parts import (attention, block, delta_rule, diff_attention, experts, latent_attention, mlp, mlstm, norm, rope,  # noqa: F401
                                      selective_scan, ssm, wkv)
 
 

@@ -14,7 +14,7 @@ from dataclasses import dataclass
 from typing import Any, Dict, Tuple
 
 from lily_b200.parts.base import Block, BlockSpec, BuildContext, RunSlots, TensorSpec, build_part, register_part
-from lily_b200.parts.norm import NormedDelta, enter_stream
+from lily_b200.parts.norm import enter_stream
 
 
 @register_part("block", "prenorm")
@@ -122,7 +122,7 @@ class ParallelBlock(Block):
 class SandwichBlockSpec:
     """A norm ahead of and behind each sublayer: ``r += mult * norm_1b(mixer(norm_1(r)))``, then, where the block has a
     feed-forward, ``r += mult * norm_2b(ff(norm_2(r)))``.  The norm behind a sublayer and the add are folded into the
-    pass of the norm that comes next (``NormedDelta``), in this block or in the one after it.
+    pass of the norm that comes next (``NormedDelta``, ``TanhDelta``), in this block or in the one after it.
     ``post_divides`` False: what stands behind a sublayer is a gain per column alone (a layer scale,
     ``r += mult * gain_1b * mixer(norm_1(r))``), named like the norms behind the sublayers and folded the same way."""
 
@@ -155,7 +155,7 @@ class SandwichBlock(Block):
             self.norm_ff_post = build_part("norm", spec.norm, f"{p}.{n2b}", ctx)
             self.feed_forward = build_part("feed_forward", spec.feed_forward, f"{p}.{spec.feed_forward_name}", ctx)
             self.parts += (self.norm_ff, self.norm_ff_post, self.feed_forward)
-        self.post_gains = []
+        self.behind = []                          # of the mixer and of the feed-forward: output -> pending delta
 
     def tensors(self) -> Dict[str, TensorSpec]:
         out: Dict[str, TensorSpec] = {}
@@ -166,17 +166,15 @@ class SandwichBlock(Block):
     def load(self, get) -> None:
         for part in self.parts:
             part.load(get)
-        # the gains of the norms behind the sublayers enter a float32 sum
-        self.post_gains = [n.weight.float().contiguous() for n in (self.norm_in_post, self.norm_ff_post) if n is not None]
+        self.behind = [n.behind(self.spec.mult, self.spec.post_divides) for n in (self.norm_in_post, self.norm_ff_post) if n is not None]
 
     def forward(self, residual, delta, batch, run: RunSlots):
-        eps, mult, divides = self.spec.norm.eps, float(self.spec.mult), self.spec.post_divides
         h = self.norm_in.forward(residual, delta, delta_bias=run.stream_bias)
-        a = NormedDelta(self.mixer.forward(h, batch, run.caches[0], run.states[0], run.write_cache), self.post_gains[0], eps, mult, divides)
+        a = self.behind[0](self.mixer.forward(h, batch, run.caches[0], run.states[0], run.write_cache))
         if self.feed_forward is None:
             return a
         h = self.norm_ff.forward(residual, a)
-        return NormedDelta(self.feed_forward.forward(h, batch), self.post_gains[1], eps, mult, divides)
+        return self.behind[1](self.feed_forward.forward(h, batch))
 
 
 @dataclass(frozen=True)
@@ -211,7 +209,7 @@ class PostNormBlock(Block):
             self.norm_ff = build_part("norm", spec.norm, f"{p}.{spec.norm_names[1]}", ctx)
             self.feed_forward = build_part("feed_forward", spec.feed_forward, f"{p}.{spec.feed_forward_name}", ctx)
             self.parts += (self.norm_ff, self.feed_forward)
-        self.gains = []
+        self.behind = []
 
     def tensors(self) -> Dict[str, TensorSpec]:
         out: Dict[str, TensorSpec] = {}
@@ -222,13 +220,13 @@ class PostNormBlock(Block):
     def load(self, get) -> None:
         for part in self.parts:
             part.load(get)
-        self.gains = [n.weight.float().contiguous() for n in (self.norm_mixer, self.norm_ff) if n is not None]
+        self.behind = [n.behind(self.spec.mult) for n in (self.norm_mixer, self.norm_ff) if n is not None]
 
     def forward(self, residual, delta, batch, run: RunSlots):
-        ops, eps, mult = self.ctx.ops, self.spec.norm.eps, float(self.spec.mult)
+        ops = self.ctx.ops
         x = enter_stream(ops, residual, delta, self.ctx.dtype, run.stream_bias)
-        a = NormedDelta(self.mixer.forward(x, batch, run.caches[0], run.states[0], run.write_cache), self.gains[0], eps, mult)
+        a = self.behind[0](self.mixer.forward(x, batch, run.caches[0], run.states[0], run.write_cache))
         if self.feed_forward is None:
             return a
         x = enter_stream(ops, residual, a, self.ctx.dtype)
-        return NormedDelta(self.feed_forward.forward(x, batch), self.gains[1], eps, mult)
+        return self.behind[1](self.feed_forward.forward(x, batch))

@@ -1,16 +1,19 @@
-"""A routed mixture of small gated feed-forward layers, some of whose router outputs may stand for the identity.
+"""A routed mixture of small feed-forward layers, some of whose router outputs may stand for the identity.
 
 The router scores ``s = softmax(W_router h)`` over all its outputs, or each output by itself, ``s = sigmoid(W_router h)``
-(logits and scores in float32).  The ``top`` outputs with the largest ``s`` (``+ correction``) are chosen; their weights are
+(logits and scores in float32).  The ``top`` outputs with the largest ``s`` (``+ correction``) are chosen, with ``groups`` only
+among those of the ``keep_groups`` best of that many equal runs of neighbouring outputs (a run's score is the sum of its two
+largest choice scores); their weights are
 their scores ``s`` (without the correction), divided by the sum of the chosen scores where the spec renormalises.  The first
 ``experts`` outputs name experts with weights of their own,
 
     y = W_down (g * sigmoid(alpha g) * (u + 1)),   g = min(W_gate h, limit),   u = clamp(W_up h, -limit, limit),
 
-or, with ``activation`` "silu", ``y = W_down (silu(W_gate h) * W_up h)``; the last ``identity`` outputs name experts without
+or, with ``activation`` "silu", ``y = W_down (silu(W_gate h) * W_up h)``, or, ungated, with "relu2",
+``y = W_down max(W_up h, 0)^2``; the last ``identity`` outputs name experts without
 tensors whose output is ``h`` itself.  A weight multiplies the expert's output, or, with ``weight_on`` "input", its input:
 ``sum_e expert_e(w_e h)``; gate and up products are linear in it, so it is applied to their results ahead of the activation
-and one gathered row serves either form.  A shared expert (a gated feed-forward of its own that every token takes) may
+and one gathered row serves either form.  A shared expert (a feed-forward of the experts' form that every token takes) may
 be added, times ``sigmoid(W_sg h)``, one number a token: ``W_sg`` is one more row of the router's product.  The sum is
 returned in float32 as one plane of partial sums for the next residual add.
 
@@ -28,7 +31,7 @@ from typing import Dict, Optional, Tuple
 import torch
 
 from lily_b200.parts.base import BuildContext, FeedForward, TensorSpec, build_part, register_part
-from lily_b200.parts.mlp import SwiGLUSpec
+from lily_b200.parts.mlp import DenseMLPSpec, SwiGLUSpec
 
 
 @dataclass(frozen=True)
@@ -43,9 +46,11 @@ class RoutedExpertsSpec:
     scores: str = "softmax"       # "softmax" over all outputs | "sigmoid" of each
     correction: bool = True       # a number an output that is added to its score for the choice alone
     renormalise: bool = True      # the chosen weights are divided by their sum
-    activation: str = "swish_clamped"     # of the experts: "swish_clamped" | "silu"
+    activation: str = "swish_clamped"     # of the experts: "swish_clamped" | "silu" | "relu2" (ungated)
     weight_on: str = "output"     # what a weight multiplies: the expert's "output" | its "input"
     shared_size: int = 0          # intermediate size of the shared expert; 0: none
+    groups: int = 0               # equal runs of neighbouring outputs of which the best ``keep_groups`` can be chosen from; 0: none
+    keep_groups: int = 0
     kind: str = "routed_experts"
     # names under the part's prefix: the router, its correction, the pattern of an expert's prefix, the shared expert's
     # prefix and its gate's row
@@ -58,6 +63,10 @@ class RoutedExpertsSpec:
         return dict(self.names or ()).get(role, dict(self._DEFAULTS)[role])
 
     @property
+    def gated(self) -> bool:
+        return self.activation != "relu2"
+
+    @property
     def outputs(self) -> int:
         return self.experts + self.identity
 
@@ -67,15 +76,21 @@ class RoutedExperts(FeedForward):
     def __init__(self, spec: RoutedExpertsSpec, prefix: str, ctx: BuildContext):
         if spec.experts < 0 or spec.identity < 0 or not 1 <= spec.top <= spec.outputs:
             raise ValueError(f"top {spec.top} of {spec.experts} experts and {spec.identity} identity outputs")
-        if spec.scores not in ("softmax", "sigmoid") or spec.activation not in ("swish_clamped", "silu") or spec.weight_on not in ("output", "input"):
+        if spec.scores not in ("softmax", "sigmoid") or spec.activation not in ("swish_clamped", "silu", "relu2") or spec.weight_on not in ("output", "input"):
             raise ValueError(f"routed experts: scores {spec.scores!r}, activation {spec.activation!r}, weight on the {spec.weight_on!r}")
         if spec.weight_on == "input" and spec.identity:
             raise ValueError("a weight on the input has no place in an output that stands for the identity")
+        if spec.groups > 1 and (spec.outputs % spec.groups or not 1 <= spec.keep_groups <= spec.groups
+                                or spec.top > spec.keep_groups * (spec.outputs // spec.groups)):
+            raise ValueError(f"top {spec.top} of the best {spec.keep_groups} of {spec.groups} groups of {spec.outputs} outputs")
         self.spec, self.prefix, self.ctx = spec, prefix, ctx
         self.router = self.correction = self.w_gate_up = self.w_down = None
-        self.shared = None if not spec.shared_size else build_part(
-            "feed_forward", SwiGLUSpec(spec.hidden_size, spec.shared_size, names=tuple((r, spec.name(r)) for r in ("gate", "up", "down"))),
-            f"{prefix}.{spec.name('shared')}", ctx)
+        self.shared = None
+        if spec.shared_size:
+            names = tuple((r, spec.name(r)) for r in ("gate", "up", "down"))
+            form = SwiGLUSpec(spec.hidden_size, spec.shared_size, names=names) if spec.gated else \
+                DenseMLPSpec(spec.hidden_size, spec.shared_size, activation=spec.activation, names=names)
+            self.shared = build_part("feed_forward", form, f"{prefix}.{spec.name('shared')}", ctx)
         self.parts = () if self.shared is None else (self.shared,)
 
     def _expert(self, e: int, role: str) -> str:
@@ -90,7 +105,8 @@ class RoutedExperts(FeedForward):
             out.update(self.shared.tensors())
             out[f"{p}.{s.name('shared_gate')}"] = TensorSpec((1, s.hidden_size))
         for e in range(s.experts):
-            out[self._expert(e, "gate")] = TensorSpec((s.intermediate_size, s.hidden_size))
+            if s.gated:
+                out[self._expert(e, "gate")] = TensorSpec((s.intermediate_size, s.hidden_size))
             out[self._expert(e, "up")] = TensorSpec((s.intermediate_size, s.hidden_size))
             out[self._expert(e, "down")] = TensorSpec((s.hidden_size, s.intermediate_size))
         return out
@@ -108,20 +124,22 @@ class RoutedExperts(FeedForward):
             self.router = torch.cat([self.router, self.router.new_zeros(-self.router.shape[0] % 8, s.hidden_size)], 0).contiguous()
         ff, h = s.intermediate_size, s.hidden_size
         if s.experts:
-            first = get(self._expert(0, "gate"))
-            self.w_gate_up = torch.empty((s.experts, 2 * ff, h), dtype=first.dtype, device=first.device)
+            first = get(self._expert(0, "up"))
+            self.w_gate_up = torch.empty((s.experts, 2 * ff if s.gated else ff, h), dtype=first.dtype, device=first.device)
             self.w_down = torch.empty((s.experts, h, ff), dtype=first.dtype, device=first.device)
             for e in range(s.experts):
-                self.w_gate_up[e, :ff].copy_(get(self._expert(e, "gate")))
-                self.w_gate_up[e, ff:].copy_(get(self._expert(e, "up")))
+                if s.gated:
+                    self.w_gate_up[e, :ff].copy_(get(self._expert(e, "gate")))
+                self.w_gate_up[e, -ff:].copy_(get(self._expert(e, "up")))
                 self.w_down[e].copy_(get(self._expert(e, "down")))
         else:
             self.w_gate_up = self.w_down = torch.empty((0,), dtype=self.ctx.dtype, device=self.router.device)
 
     def forward(self, x, batch):
         s, ops = self.spec, self.ctx.ops
+        grouped = {"groups": s.groups, "keep_groups": s.keep_groups} if s.groups > 1 else {}
         routing = ops.moe_route(x, self.router, self.correction, s.top, s.experts, scores=s.scores, renormalise=s.renormalise,
-                                shared_gate=self.shared is not None, outputs=s.outputs)
+                                shared_gate=self.shared is not None, outputs=s.outputs, **grouped)
         shared = None if self.shared is None else self.shared.forward(x, batch)
         out = ops.moe_experts(x, routing, self.w_gate_up, self.w_down, s.limit, s.alpha, activation=s.activation,
                               weight_on_input=s.weight_on == "input", shared=shared)

@@ -1,9 +1,12 @@
-"""RMSNorm fused with the residual add.
+"""Norms fused with the residual add: RMSNorm, and a norm that squashes instead of dividing (``DynamicTanh``).
 
 ``forward(residual, delta)`` adds ``delta`` into the float32 residual stream in place and
 returns the normalised activations in the compute dtype: the fused-add convention of
 lily/layers/layernorm.py:11-47 with the sum kept in float32.  With ``rows`` only those rows are
 normalised (the final norm before the logits).
+
+A norm may also stand behind a sublayer: ``behind(mult)`` gives what turns the sublayer's output into a pending delta
+(``NormedDelta``, ``TanhDelta``) that the norm which comes next folds into the stream in its own pass.
 """
 
 from __future__ import annotations
@@ -25,6 +28,21 @@ class NormedDelta:
     eps: float
     mult: float = 1.0
     normalise: bool = True     # False: ``mult * (delta * gain)``, a gain per column without the division (a layer scale)
+
+
+@dataclass
+class TanhDelta:
+    """A sublayer's output that enters the residual stream as ``mult * (gain * tanh(alpha * delta) + shift)``."""
+
+    delta: Any                 # as in ``NormedDelta``
+    alpha: float
+    gain: Any                  # float32 [size]
+    shift: Any                 # float32 [size]
+    mult: float = 1.0
+
+    @property
+    def norm(self):
+        return self.alpha, self.gain, self.shift
 
 
 @dataclass(frozen=True)
@@ -54,9 +72,17 @@ class RMSNorm(Norm):
         if self.spec.single_gain:
             self.weight = self.weight.float().reshape(1).expand(self.spec.size).contiguous()      # the kernels read a gain a column
 
+    def behind(self, mult: float = 1.0, divides: bool = True):
+        """What a block wraps a sublayer's output in when this norm stands behind the sublayer (``divides`` False: its gain alone)."""
+        gain = self.weight.float().contiguous()                  # it enters a float32 sum
+        return lambda delta: NormedDelta(delta, gain, self.spec.eps, float(mult), divides)
+
     def forward(self, residual, delta=None, delta_bias=None, rows=None, write_residual=True, also=None, out_dtype=None):
         """``delta`` may be a tuple of tensors to be summed; ``delta_bias`` a float32 vector added to every row;
         ``also`` another norm of this kind and size whose output of the same rows is wanted too (returns a pair)."""
+        if isinstance(delta, TanhDelta):
+            self.ctx.ops.add_tanh_norm(residual, delta.delta, delta.norm, delta.mult, None, None)
+            delta = None
         if isinstance(delta, NormedDelta):
             if delta_bias is not None or also is not None:
                 raise ValueError("a normalised delta comes alone: no stream vector and no second norm in the same pass")
@@ -80,13 +106,78 @@ class RMSNorm(Norm):
         return outs if also is not None else outs[0]
 
 
+@dataclass(frozen=True)
+class DynamicTanhSpec:
+    """``gain * tanh(alpha * x) + shift``: a scalar ``alpha``, a gain and a shift a column; no mean and no variance."""
+
+    size: int
+    kind: str = "dynamic_tanh"
+    suffix: str = ""               # the gain's, the scalar's and the shift's names are the part's prefix followed by these
+    alpha_suffix: str = ".alpha"
+    shift_suffix: str = ".b"
+
+
+@register_part("norm", "dynamic_tanh")
+class DynamicTanh(Norm):
+    def __init__(self, spec: DynamicTanhSpec, prefix: str, ctx: BuildContext):
+        self.spec, self.prefix, self.ctx = spec, prefix, ctx
+        self.alpha = 0.0
+        self.weight = self.shift = None
+
+    def tensors(self) -> Dict[str, TensorSpec]:
+        s, p = self.spec, self.prefix
+        return {f"{p}{s.suffix}": TensorSpec((s.size,), role="vector", init="gain"),
+                f"{p}{s.alpha_suffix}": TensorSpec((), role="vector", init="half"),
+                f"{p}{s.shift_suffix}": TensorSpec((s.size,), role="vector", init="zeros")}
+
+    def load(self, get) -> None:
+        s, p = self.spec, self.prefix
+        # every column enters float32 arithmetic; the scalar travels as a kernel argument
+        self.alpha = float(get(f"{p}{s.alpha_suffix}").float().item())
+        self.weight = get(f"{p}{s.suffix}").float().contiguous()
+        self.shift = get(f"{p}{s.shift_suffix}").float().contiguous()
+
+    @property
+    def norm(self):
+        return self.alpha, self.weight, self.shift
+
+    def behind(self, mult: float = 1.0, divides: bool = True):
+        if not divides:
+            raise ValueError("a norm that squashes has no form with the gain alone")
+        return lambda delta: TanhDelta(delta, self.alpha, self.weight, self.shift, float(mult))
+
+    def forward(self, residual, delta=None, delta_bias=None, rows=None, write_residual=True, also=None, out_dtype=None):
+        ops, dtype = self.ctx.ops, out_dtype or self.ctx.dtype
+        if also is not None:
+            raise ValueError("this norm shares no pass with another norm of the same rows")
+        post, mult = None, 1.0
+        if isinstance(delta, TanhDelta):
+            post, mult, delta = delta.norm, delta.mult, delta.delta
+        elif isinstance(delta, NormedDelta):
+            ops.add_normed(residual, delta.delta, delta.gain, delta.eps, delta.mult, residual.dtype,
+                           **({} if delta.normalise else {"normalise": False}))
+            delta = None
+        elif isinstance(delta, (tuple, list)):
+            deltas = [d for d in delta if d is not None]
+            delta = deltas[0] if deltas else None
+            if len(deltas) > 1:
+                ops.add_rmsnorm_multi(residual, deltas, [], 1.0, dtype)
+                delta = None
+        if delta_bias is not None:
+            ops.add_rmsnorm_multi(residual, [], [], 1.0, dtype, bias=delta_bias)
+        return ops.add_tanh_norm(residual, delta, post, mult, self.norm, dtype, rows=rows, write_residual=write_residual and rows is None)
+
+
 def enter_stream(ops, residual, delta, dtype, bias=None):
     """Adds a pending ``delta`` (a tensor, several of them, a ``NormedDelta`` or None) and ``bias`` (a row vector) into the
     float32 stream in place and returns the new stream itself in ``dtype``: what a sublayer takes that has no norm ahead
     of it.  With ``dtype`` float32 that is ``residual``, which the next call changes."""
+    if isinstance(delta, (NormedDelta, TanhDelta)) and bias is not None:
+        raise ValueError("a normalised delta comes alone: no stream vector in the same pass")
+    if isinstance(delta, TanhDelta):
+        out = ops.add_tanh_norm(residual, delta.delta, delta.norm, delta.mult, None, None if dtype == residual.dtype else dtype)
+        return residual if out is None else out
     if isinstance(delta, NormedDelta):
-        if bias is not None:
-            raise ValueError("a normalised delta comes alone: no stream vector in the same pass")
         return ops.add_normed(residual, delta.delta, delta.gain, delta.eps, delta.mult, dtype,
                               **({} if delta.normalise else {"normalise": False}))
     deltas = [d for d in delta if d is not None] if isinstance(delta, (tuple, list)) else ([delta] if delta is not None else [])

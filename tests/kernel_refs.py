@@ -117,14 +117,16 @@ def _pages(kv_layer, nkv, page_size, d, dv, values_in_keys=False):
 
 
 def qk_norm_rope_write(qkv, q_gain, k_gain, eps, cos, sin, positions, token_req, block_table, kv_layer, nq, nkv, d,
-                       rotary_dim, page_size, write_kv=True, q_out=None, dv=None, v_norm=False, v_keep=None, v_blend=None):
+                       rotary_dim, page_size, write_kv=True, q_out=None, dv=None, v_norm=False, v_keep=None, v_blend=None, row=None):
     qkv = _sum(qkv)
     n = qkv.shape[0]
     dv = dv or d
     x = qkv.float()
-    q = x[:, :nq * d].view(n, nq, d)
-    k = x[:, nq * d:(nq + nkv) * d].view(n, nkv, d)
-    v = x[:, (nq + nkv) * d:].view(n, nkv, dv)
+    assert x.shape[1] == (row or (nq + nkv) * d + nkv * dv)
+    q = x[:, :nq * d].reshape(n, nq, d)
+    if write_kv:
+        k = x[:, nq * d:(nq + nkv) * d].reshape(n, nkv, d)
+        v = x[:, (nq + nkv) * d:(nq + nkv) * d + nkv * dv].reshape(n, nkv, dv)
 
     def norm(t, gain):
         if gain is None:
@@ -267,10 +269,10 @@ def _gather_kv(kv_layer, table_row, length, page_size, nkv=None, d=None, dv=None
     return k.float(), v.float()
 
 
-def _attend(q, k, v, q_pos, scale, window, softcap=None, keep_first=0, sink=False, all_values=False):
+def _attend(q, k, v, q_pos, scale, window, softcap=None, keep_first=0, sink=False, all_values=False, sinks=None):
     """q [rows, nq, d] at positions q_pos [rows]; k [keys, nkv, d], v [keys, nkv, dv] at positions 0..keys-1.
     ``sink``: a key of score 0 without a value joins the softmax; ``all_values``: every query head's weights over the
-    values of every kv head, [rows, nq, nkv * dv]."""
+    values of every kv head, [rows, nq, nkv * dv]; ``sinks`` [nq]: such a key with a score of the head's own."""
     rep = q.shape[1] // k.shape[1]
     kk, vv = k.repeat_interleave(rep, 1), v.repeat_interleave(rep, 1)
     s = torch.einsum("qhd,khd->hqk", q, kk) * scale
@@ -281,8 +283,9 @@ def _attend(q, k, v, q_pos, scale, window, softcap=None, keep_first=0, sink=Fals
     if window:
         seen &= (kpos[None, :] > q_pos[:, None] - window) | (kpos[None, :] < keep_first)
     s = s.masked_fill(~seen[None], float("-inf"))
-    if sink:
-        p = torch.softmax(torch.cat([s, torch.zeros_like(s[..., :1])], -1), -1)[..., :-1]
+    if sink or sinks is not None:
+        unit = torch.zeros_like(s[..., :1]) if sinks is None else sinks.float()[:, None, None].expand_as(s[..., :1])
+        p = torch.softmax(torch.cat([s, unit], -1), -1)[..., :-1]
     else:
         p = torch.softmax(s, -1)
     if all_values:
@@ -292,44 +295,51 @@ def _attend(q, k, v, q_pos, scale, window, softcap=None, keep_first=0, sink=Fals
 
 def attention_prefill(q, kv_layer, block_table, cu_seqlens, prefix_lens, tile_req, tile_start, out, nq, nkv, d,
                       page_size, scale, window=None, tile_rows=None, heads_per_block=0, softcap=None, dv=None,
-                      values_in_keys=False, keep_first=0, sink=False, all_values=False):
+                      values_in_keys=False, keep_first=0, sink=False, all_values=False, sinks=None):
     dv = dv or d
     for r in sorted(set(tile_req.tolist())):
         t0, t1 = int(cu_seqlens[r]), int(cu_seqlens[r + 1])
         prefix = int(prefix_lens[r])
         k, v = _gather_kv(kv_layer, block_table[r], prefix + t1 - t0, page_size, nkv, d, dv, values_in_keys)
         qpos = torch.arange(prefix, prefix + t1 - t0, device=q.device)
-        o = _attend(q[t0:t1].float().view(-1, nq, d), k, v, qpos, scale, window, softcap, keep_first, sink, all_values)
+        o = _attend(q[t0:t1].float().view(-1, nq, d), k, v, qpos, scale, window, softcap, keep_first, sink, all_values, sinks)
         out[t0:t1] = o.reshape(t1 - t0, -1).to(out.dtype)
 
 
 def attention_decode(q, kv_layer, block_table, seq_lens, out, scratch, splits, nq, nkv, d, page_size, scale,
                      window=None, stages=0, softcap=None, dv=None, values_in_keys=False, keep_first=0, sink=False,
-                     all_values=False):
+                     all_values=False, sinks=None):
     dv = dv or d
     for r in range(q.shape[0]):
         n = int(seq_lens[r])
         k, v = _gather_kv(kv_layer, block_table[r], n, page_size, nkv, d, dv, values_in_keys)
         o = _attend(q[r:r + 1].float().view(1, nq, d), k, v, torch.tensor([n - 1], device=q.device), scale, window, softcap,
-                    keep_first, sink, all_values)
+                    keep_first, sink, all_values, sinks)
         out[r] = o.reshape(-1).to(out.dtype)
 
 
 def attention_decode_fused(qkv, q_gain, k_gain, eps, cos, sin, kv_layer, block_table, seq_lens, out, scratch, splits, nq, nkv,
-                           d, rotary_dim, page_size, scale, window=None, write_kv=True, stages=0, softcap=None):
+                           d, rotary_dim, page_size, scale, window=None, write_kv=True, stages=0, softcap=None, row=None):
     """What the one kernel does, as the two statements it replaces: every request brings one token, at position
     seq_len - 1."""
     qkv = _sum(qkv)
     n = qkv.shape[0]
     q = qk_norm_rope_write(qkv, q_gain, k_gain, eps, cos, sin, (seq_lens - 1).to(torch.int32),
                            torch.arange(n, dtype=torch.int32, device=qkv.device), block_table, kv_layer, nq, nkv, d, rotary_dim,
-                           page_size, write_kv=write_kv)
+                           page_size, write_kv=write_kv, row=row)
     attention_decode(q.to(out.dtype), kv_layer, block_table, seq_lens, out, scratch, splits, nq, nkv, d, page_size, scale, window,
                      softcap=softcap)
 
 
 def sigmoid_gate(out, gate):
     out.copy_((out.float() * torch.sigmoid(_sum(gate).float())).to(out.dtype))
+    return out
+
+
+def sigmoid_head_gate(out, gate, g0, heads):
+    n, cols = out.shape
+    g = torch.sigmoid(_sum(gate).float()[:, g0:g0 + heads])
+    out.copy_((out.float().view(n, heads, cols // heads) * g[:, :, None]).view(n, cols).to(out.dtype))
     return out
 
 
@@ -551,7 +561,7 @@ def latent_prepare(down, q0, q_rank, kv0, rank, rot, rotary_dim, q_gain, kv_gain
                    block_table, layer, page_size, write_kv=True):
     x = _sum(down).float()
     unit = lambda t: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
-    cq = (unit(x[:, q0:q0 + q_rank]) * q_gain.float()).to(layer.dtype)
+    cq = (unit(x[:, q0:q0 + q_rank]) * q_gain.float()).to(layer.dtype) if q_rank else None
     if write_kv:
         latent = unit(x[:, kv0:kv0 + rank]) * kv_gain.float()
         turned = _rotate_halves(x[:, kv0 + rank:kv0 + rank + rot], cos, sin, positions, rotary_dim)
@@ -583,13 +593,20 @@ class ExpertRouting:
     gate: Optional[torch.Tensor] = None
 
 
-def moe_route(h, router, correction, top, experts, scores="softmax", renormalise=True, shared_gate=False, outputs=None):
+def moe_route(h, router, correction, top, experts, scores="softmax", renormalise=True, shared_gate=False, outputs=None, groups=0,
+              keep_groups=0):
     z = h.float() @ router.float().t()
     outputs = router.shape[0] - int(shared_gate) if outputs is None else outputs
     gate = torch.sigmoid(z[:, outputs]) if shared_gate else None
     z = z[:, :outputs]
     s = torch.softmax(z, -1) if scores == "softmax" else torch.sigmoid(z)
-    chosen = torch.topk(s if correction is None else s + correction.float(), top, dim=-1).indices
+    choice = s if correction is None else s + correction.float()
+    if groups > 1:
+        runs = choice.view(len(s), groups, -1)
+        best = runs.topk(min(2, runs.shape[-1]), dim=-1).values.sum(-1)
+        out_of = torch.ones_like(best, dtype=torch.bool).scatter_(1, best.topk(keep_groups, dim=-1).indices, False)
+        choice = runs.masked_fill(out_of[..., None], float("-inf")).reshape(len(s), -1)
+    chosen = torch.topk(choice, top, dim=-1).indices
     picked = torch.gather(s, 1, chosen)
     if renormalise:
         picked = picked / (picked.sum(-1, keepdim=True) + 1e-20)
@@ -607,7 +624,9 @@ def moe_experts(h, routing, w_gate_up, w_down, limit=0.0, alpha=0.0, activation=
             if e < experts:
                 gu = w_gate_up[e].float() @ (a * x[t] if weight_on_input else x[t])
                 g, u = gu[:ff], gu[ff:]
-                if activation == "silu":
+                if activation == "relu2":
+                    act = torch.clamp(gu, min=0) ** 2
+                elif activation == "silu":
                     act = g * torch.sigmoid(g) * u
                 else:
                     g, u = g.clamp(max=limit), u.clamp(min=-limit, max=limit)
@@ -645,6 +664,22 @@ def add_normed_rmsnorm(resid, delta, post_gain, post_eps, mult, weight, eps, out
 def add_normed(resid, delta, post_gain, post_eps, mult, out_dtype, normalise=True):
     add_normed_rmsnorm(resid, delta, post_gain, post_eps, mult, None, 1.0, out_dtype, normalise=normalise)
     return resid.to(out_dtype)
+
+
+def add_tanh_norm(resid, delta, post, mult, pre, out_dtype, rows=None, write_residual=True):
+    v = resid
+    if delta is not None:
+        d = _sum(delta).float()
+        if post is not None:
+            d = torch.tanh(post[0] * d) * post[1] + post[2]
+        v = resid + mult * d
+    if rows is not None:
+        v = v[rows.long()]
+    elif write_residual and delta is not None:
+        resid.copy_(v)
+    if out_dtype is None:
+        return None
+    return (v if pre is None else torch.tanh(pre[0] * v) * pre[1] + pre[2]).to(out_dtype)
 
 
 def _activate(z, activation, factors=(0.0, 0.0)):
@@ -788,3 +823,54 @@ def selective_scan(x, low, b_col, step, proj, z_col, a, d_skip, state, cu_seqlen
         if t1 > t0:
             row[:inner * n] = S.reshape(-1)
     return out.to(x.dtype)
+
+
+# ---------------------------------------------------------------------------- matrix memory with exponential gates
+
+def mlstm_max_head_dim():
+    return 512
+
+
+MLSTM_CHUNK = 64
+
+
+def mlstm_plan(new_lens, dtype, d, dv, device):
+    return None
+
+
+def mlstm_workspace_floats(plan, heads, d, dv):
+    return 0
+
+
+def mlstm_scan(proj, q_col, k_col, v_col, gates, i_col, f_col, i_bias, f_bias, cap, q_scale, state, cu_seqlens, slots, requests, heads,
+               d, dv, plan=None, workspace=None):
+    x, z = _sum(proj).float(), _sum(gates).float()
+    n = x.shape[0]
+    q = x[:, q_col:q_col + heads * d].reshape(n, heads, d) * q_scale
+    k = x[:, k_col:k_col + heads * d].reshape(n, heads, d)
+    v = torch.cat([x[:, v_col:v_col + heads * dv].reshape(n, heads, dv), torch.ones(n, heads, 1)], -1)
+    soft = lambda t: cap * torch.tanh(t / cap)
+    i = soft(z[:, i_col:i_col + heads] + i_bias)
+    f = torch.nn.functional.logsigmoid(soft(z[:, f_col:f_col + heads] + f_bias))
+    out, scale = torch.zeros(n, heads, dv + 1), torch.zeros(n, heads)
+    size = heads * (dv + 1) * d
+    for r in range(requests):
+        row = state[int(slots[r])]
+        S, m = row[:size].view(heads, dv + 1, d), row[size:size + heads].clone()
+        for t in range(int(cu_seqlens[r]), int(cu_seqlens[r + 1])):
+            new = torch.maximum(f[t] + m, i[t])
+            keep, write = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
+            S.copy_(keep[:, None, None] * S + torch.einsum("h,hj,hi->hji", write, v[t], k[t]))
+            out[t] = torch.einsum("hji,hi->hj", S, q[t])
+            scale[t] = m = new
+    return out[..., :dv].reshape(n, heads * dv).contiguous(), out[..., dv].contiguous(), scale
+
+
+def mlstm_out(y, nq, m, gate, gate_col, gain, floor, eps, state, m_off, cu_seqlens, token_req, slots, out_dtype):
+    n, heads = nq.shape
+    o = y.view(n, heads, -1) / (torch.maximum(nq.abs(), torch.exp(-m)) + floor)[..., None]
+    o = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)).reshape(n, -1)
+    for r in range(len(slots)):
+        last = int(cu_seqlens[r + 1]) - 1
+        state[int(slots[r]), m_off:m_off + heads] = m[last]
+    return (o * gain * torch.sigmoid(_sum(gate).float()[:, gate_col:gate_col + y.shape[1]])).to(out_dtype)
