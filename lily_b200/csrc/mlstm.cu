@@ -11,6 +11,7 @@
 //
 //   mlstm_scan   raw sums S^T q_t [tokens, heads, dv], n . q_t [tokens, heads] and m_t [tokens, heads]: a block owns a few
 //                columns of one head of one request and walks the request's new tokens in order
+//                (long portions in bfloat16 run in chunks side by side instead: mlstm_chunk.cu)
 //   mlstm_out    the division, each head's unit root mean square, gain and sigmoid gate; writes the last token's m into the
 //                slot (every block of the scan reads the old one)
 //

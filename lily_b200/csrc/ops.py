@@ -48,6 +48,8 @@ _SIGNATURES = {
     "lily_add_tanh_norm": [_vp, _vp, _i, _i, _sz, _f, _vp, _vp, _f, _f, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _vp],
     "lily_mlstm_scan": [_vp, _i, _i, _sz, _i, _i, _i, _i, _vp, _i, _i, _sz, _i, _i, _i, _vp, _vp, _f, _f, _vp, _sz, _vp, _vp, _vp, _vp, _vp,
                         _vp, _i, _i, _i, _i, _vp],
+    "lily_mlstm_chunks": [_vp, _i, _i, _i, _i, _vp, _i, _i, _sz, _i, _i, _i, _vp, _vp, _f, _f, _vp, _sz, _vp, _vp, _vp, _vp, _vp, _vp, _vp,
+                          _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _vp, _i, _i, _i, _i, _vp],
     "lily_mlstm_out": [_vp, _vp, _vp, _vp, _i, _i, _sz, _i, _i, _vp, _f, _f, _vp, _i, _vp, _sz, _sz, _vp, _vp, _vp, _i, _i, _i, _vp],
     "lily_normed_mean": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _sz, _vp, _i, _i, _f, _f, _vp],
     "lily_causal_conv_silu": [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _sz, _sz, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _vp],
@@ -144,6 +146,10 @@ def library():
         lib.lily_delta_rule_max_head_dim.restype = _i
         lib.lily_selective_scan_max_state.restype = _i
         lib.lily_mlstm_max_head_dim.restype = _i
+        lib.lily_mlstm_chunk_takes.argtypes = [_i, _i]
+        lib.lily_mlstm_chunk_takes.restype = _i
+        lib.lily_mlstm_chunk_floats.argtypes = [_i, _i, _i, _i, _i]
+        lib.lily_mlstm_chunk_floats.restype = _sz
         _lib = lib
     return _lib
 
@@ -1947,13 +1953,72 @@ def mlstm_max_head_dim() -> int:
     return int(library().lily_mlstm_max_head_dim())
 
 
+MLSTM_CHUNK = 128        # tokens a chunk of a long portion (doubled while the chunks' states would pass SCAN_WORKSPACE)
+MLSTM_DIRECT = 64        # portions up to this many tokens run in one piece, from and to the state in the slot
+MLSTM_TILE = 64          # tokens a tile of the chunk kernels
+
+
+@dataclass
+class MlstmPlan:
+    """How a step's recurrence over matrix memories is cut: the portions that run in one piece (``direct``), and the long ones in
+    chunks side by side with their tiles of ``MLSTM_TILE`` tokens.  All lists are int32 on the device."""
+
+    direct: torch.Tensor
+    num_direct: int
+    item_req: torch.Tensor
+    item_start: torch.Tensor
+    item_len: torch.Tensor
+    items: int
+    long_req: torch.Tensor
+    long_first: torch.Tensor
+    long_count: torch.Tensor
+    longs: int
+    tile_item: torch.Tensor
+    tile_start: torch.Tensor
+    tiles: int
+    tokens: int                              # of the whole step
+
+
+def mlstm_plan(new_lens: Sequence[int], dtype: torch.dtype, heads: int, d: int, dv: int, device) -> Optional[MlstmPlan]:
+    """None when every portion runs in one piece: portions of up to ``MLSTM_DIRECT`` tokens, float32, and head sizes the chunk
+    kernels do not take (keys not a multiple of 16, values not of 8)."""
+    longs = [r for r, n in enumerate(new_lens) if n > MLSTM_DIRECT]
+    if not longs or dtype != torch.bfloat16 or not library().lily_mlstm_chunk_takes(int(d), int(dv)):
+        return None
+    chunk, state = MLSTM_CHUNK, 8 * heads * dv * d
+    while chunk < 2048 and sum(-(-new_lens[r] // chunk) for r in longs) * state > SCAN_WORKSPACE:
+        chunk *= 2
+    direct = [r for r, n in enumerate(new_lens) if n <= MLSTM_DIRECT]
+    req, start, length, first, count, tile_item, tile_start = [], [], [], [], [], [], []
+    for r in longs:
+        first.append(len(req))
+        for s in range(0, new_lens[r], chunk):
+            n = min(chunk, new_lens[r] - s)
+            tile_item += [len(req)] * -(-n // MLSTM_TILE)
+            tile_start += range(0, n, MLSTM_TILE)
+            req.append(r)
+            start.append(s)
+            length.append(n)
+        count.append(len(req) - first[-1])
+    flat = torch.tensor(direct + req + start + length + longs + first + count + tile_item + tile_start, dtype=torch.int32)
+    parts = torch.split(flat.to(device, non_blocking=True), [len(direct)] + [len(req)] * 3 + [len(longs)] * 3 + [len(tile_item)] * 2)
+    return MlstmPlan(parts[0], len(direct), parts[1], parts[2], parts[3], len(req), parts[4], parts[5], parts[6], len(longs), parts[7], parts[8],
+                     len(tile_item), sum(new_lens))
+
+
+def mlstm_workspace_floats(plan: Optional[MlstmPlan], heads: int, d: int, dv: int) -> int:
+    return 0 if plan is None else int(library().lily_mlstm_chunk_floats(plan.items, plan.tokens, heads, d, dv))
+
+
 def mlstm_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, gates: torch.Tensor, i_col: int, f_col: int, i_bias: torch.Tensor,
                f_bias: torch.Tensor, cap: float, q_scale: float, state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor,
-               requests: int, heads: int, d: int, dv: int) -> Tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+               requests: int, heads: int, d: int, dv: int, plan: Optional[MlstmPlan] = None,
+               workspace: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
     """The recurrence of the matrix memory over each request's new tokens, from and to ``state[slot]`` (float32, [heads, dv + 1,
     d] with the normaliser as the last column, then the heads' scales, which ``mlstm_out`` writes).  ``proj`` [tokens, width]
     holds q and k (heads x d) and v (heads x dv) from their columns on, ``gates`` [tokens, width] the gates' inputs before their
-    biases (either may be float32 partial sums).  q is multiplied by ``q_scale``.  Returns float32 (S^T q [tokens, heads * dv],
+    biases (either may be float32 partial sums).  q is multiplied by ``q_scale``.  With a ``plan`` (``mlstm_plan``) and its
+    ``workspace`` (float32, ``mlstm_workspace_floats``) the long portions of a bfloat16 ``proj`` run as chunks side by side.  Returns float32 (S^T q [tokens, heads * dv],
     n . q [tokens, heads], m [tokens, heads])."""
     _dev(proj, gates, i_bias, f_bias, state, cu_seqlens, slots)
     n, ld = proj.shape[-2:]
@@ -1965,10 +2030,22 @@ def mlstm_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, gates: to
         raise KernelError("mlstm_scan: biases [heads] and state are float32")
     y = torch.empty((n, heads * dv), dtype=torch.float32, device=proj.device)
     nm = torch.empty((2, n, heads), dtype=torch.float32, device=proj.device)
-    _call("lily_mlstm_scan", *_operand(proj, n, ld, "mlstm_scan"), ld, int(q_col), int(k_col), int(v_col),
-          *_operand(gates, n, gld, "mlstm_scan gates"), gld, int(i_col), int(f_col), _p(i_bias), _p(f_bias), float(cap), float(q_scale),
-          _p(state), state.stride(0), _p(y), nm[0].data_ptr(), nm[1].data_ptr(), _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots"), None,
-          int(requests), heads, d, dv, _stream())
+    if plan is not None and (proj.dtype != torch.bfloat16 or workspace is None):
+        plan = None                                    # a product in float32, or no scratch to be had: every portion runs whole
+    columns = (ld, int(q_col), int(k_col), int(v_col))
+    gate_args = (*_operand(gates, n, gld, "mlstm_scan gates"), gld, int(i_col), int(f_col), _p(i_bias), _p(f_bias), float(cap), float(q_scale))
+    out = (_p(state), state.stride(0), _p(y), nm[0].data_ptr(), nm[1].data_ptr(), _i32(cu_seqlens, "cu_seqlens"), _i32(slots, "slots"))
+    if plan is not None:
+        need = mlstm_workspace_floats(plan, heads, d, dv)
+        if workspace.dtype != torch.float32 or workspace.numel() < need or plan.tokens != n:
+            raise KernelError(f"mlstm_scan: chunks of {plan.tokens} tokens need a float32 workspace of {need}")
+        _call("lily_mlstm_chunks", _p(proj), *columns, *gate_args, *out, _p(plan.item_req), _p(plan.item_start), _p(plan.item_len), plan.items,
+              _p(plan.long_req), _p(plan.long_first), _p(plan.long_count), plan.longs, _p(plan.tile_item), _p(plan.tile_start), plan.tiles,
+              _p(workspace), n, heads, d, dv, _stream())
+        launches["count"] += 3                         # four kernels behind one face
+    if plan is None or plan.num_direct:
+        _call("lily_mlstm_scan", *_operand(proj, n, ld, "mlstm_scan"), *columns, *gate_args, *out, None if plan is None else _p(plan.direct),
+              int(requests) if plan is None else plan.num_direct, heads, d, dv, _stream())
     return y, nm[0], nm[1]
 
 

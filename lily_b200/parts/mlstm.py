@@ -120,9 +120,14 @@ class Mlstm(Mixer):
         s, ops = self.spec, self.ctx.ops
         proj, gates, i_col = self._project(x)
         v_col = 2 * s.key_columns
+        # long portions run as chunks side by side; the cut is planned once a step for the layers of one size
+        plan = batch.plan(("mlstm_plan", s.heads, s.head_dim, s.v_head_dim), lambda b: ops.mlstm_plan(
+            b.h_new_lens, x.dtype, s.heads, s.head_dim, s.v_head_dim, b.token_ids.device))
+        need = ops.mlstm_workspace_floats(plan, s.heads, s.head_dim, s.v_head_dim)
+        room = batch.workspace.floats("mlstm_chunks", need) if need and batch.workspace is not None else None
         y, nq, m = ops.mlstm_scan(proj, 0, s.key_columns, v_col, gates, i_col, i_col + s.heads, self.i_bias, self.f_bias, s.gate_cap,
                                   s.head_dim ** -0.5, state, batch.cu_seqlens, batch.slots, batch.num_requests, s.heads, s.head_dim,
-                                  s.v_head_dim)
+                                  s.v_head_dim, plan=plan, workspace=room)
         out = ops.mlstm_out(y, nq, m, proj, v_col + s.inner, self.gain, s.floor, s.norm_eps, state, self.matrix_floats, batch.cu_seqlens,
                             batch.token_req, batch.slots, self.ctx.dtype)
         return ops.linear_auto(out, self.w_o)

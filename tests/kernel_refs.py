@@ -831,10 +831,7 @@ def mlstm_max_head_dim():
     return 512
 
 
-MLSTM_CHUNK = 64
-
-
-def mlstm_plan(new_lens, dtype, d, dv, device):
+def mlstm_plan(new_lens, dtype, heads, d, dv, device):
     return None
 
 
