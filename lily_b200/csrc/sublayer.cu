@@ -237,14 +237,16 @@ struct TanhAddArgs {
     int write_residual;
 };
 
-// tanh z for outputs that are rounded to bfloat16 and for sums of them: its power series (to z^9: below 1e-7 of the value) within
-// a quarter of zero, else 1 - 2 / (1 + e^(2 |z|)) by the hardware's exponential and quotient, a few units of float32.
+// tanh z.  In the bfloat16 path (outputs rounded to bfloat16, and float32 sums of sublayers that were) 1 - 2 / (1 + e^(2 |z|)) by
+// the hardware's power of two and reciprocal, a few units of float32 next to one, and the power series z - z^3/3 + 2 z^5/15 (to
+// 6e-8 of the value) within a tenth of zero, where that difference would cancel.
 template <typename T> __device__ __forceinline__ float squash(float z) { return tanhf(z); }
 template <> __device__ __forceinline__ float squash<__nv_bfloat16>(float z) {
-    const float z2 = z * z, t = fabsf(z);
-    const float series = z * fmaf(z2, fmaf(z2, fmaf(z2, fmaf(z2, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
-    const float far = 1.f - __fdividef(2.f, 1.f + __expf(fminf(2.f * t, 40.f)));
-    return t < 0.25f ? series : copysignf(far, z);
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(fabsf(z) * 2.885390081777927f));      // 2 / ln 2
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+    const float z2 = z * z, series = z * fmaf(z2, fmaf(z2, 2.f / 15.f, -1.f / 3.f), 1.f);
+    return fabsf(z) < 0.1f ? series : copysignf(fmaf(-2.f, r, 1.f), z);
 }
 
 // grid (ceil(hidden / (VEC * blockDim)), ceil(rows / ROWS)): a thread owns VEC neighbouring columns of ROWS rows, so that gains
@@ -264,13 +266,13 @@ __global__ void add_tanh_norm_kernel(const TanhAddArgs a) {
     }
     float v[ROWS][VEC], d[ROWS][VEC];
 #pragma unroll
-    for (int r = 0; r < ROWS; ++r) {
-        const int m = blockIdx.y * ROWS + r;
-        if (m >= a.n_out) break;
+    for (int r = 0; r < ROWS; ++r) {                             // every row is asked for before the first is worked on
+        const int m = min((int)blockIdx.y * ROWS + r, a.n_out - 1);
         const size_t src = (size_t)(a.rows ? a.rows[m] : m) * a.hidden + i;
-        if (VEC == 4) {
-            *reinterpret_cast<float4*>(v[r]) = *reinterpret_cast<const float4*>(a.resid + src);
-            *reinterpret_cast<float4*>(d[r]) = a.delta.p ? a.delta.four(src) : make_float4(0.f, 0.f, 0.f, 0.f);
+        if constexpr (VEC == 4) {
+            const float4 x = *reinterpret_cast<const float4*>(a.resid + src), y = a.delta.p ? a.delta.four(src) : make_float4(0.f, 0.f, 0.f, 0.f);
+            v[r][0] = x.x; v[r][1] = x.y; v[r][2] = x.z; v[r][3] = x.w;
+            d[r][0] = y.x; d[r][1] = y.y; d[r][2] = y.z; d[r][3] = y.w;
         } else {
             v[r][0] = a.resid[src];
             d[r][0] = a.delta.p ? a.delta(src) : 0.f;
@@ -279,26 +281,28 @@ __global__ void add_tanh_norm_kernel(const TanhAddArgs a) {
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
         const int m = blockIdx.y * ROWS + r;
-        if (m >= a.n_out) break;
-        if (a.delta.p) {
+        if (m < a.n_out) {
+            if (a.delta.p) {
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) {
-                const float u = a.post.gain ? fmaf(squash<T>(a.post.alpha * d[r][e]), pg[e], ps[e]) : d[r][e];
-                v[r][e] = fmaf(a.mult, u, v[r][e]);
+                for (int e = 0; e < VEC; ++e) {
+                    const float u = a.post.gain ? fmaf(squash<T>(a.post.alpha * d[r][e]), pg[e], ps[e]) : d[r][e];
+                    v[r][e] = fmaf(a.mult, u, v[r][e]);
+                }
+                if (a.write_residual) {                          // every token then: row m is token m
+                    float* dst = a.resid + (size_t)m * a.hidden + i;
+                    if constexpr (VEC == 4) *reinterpret_cast<float4*>(dst) = make_float4(v[r][0], v[r][1], v[r][2], v[r][3]);
+                    else dst[0] = v[r][0];
+                }
             }
-            if (a.write_residual) {
-                float* dst = a.resid + (size_t)(a.rows ? a.rows[m] : m) * a.hidden + i;
-                if (VEC == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(v[r]);
-                else dst[0] = v[r][0];
+            if (a.out != nullptr) {
+                T* dst = (T*)a.out + (size_t)m * a.hidden + i;
+                float o[VEC];
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) o[e] = a.pre.gain ? fmaf(squash<T>(a.pre.alpha * v[r][e]), g[e], s[e]) : v[r][e];
+                if constexpr (VEC == 4) store_four<T>(dst, make_float4(o[0], o[1], o[2], o[3]));
+                else dst[0] = from_float<T>(o[0]);
             }
         }
-        if (a.out == nullptr) continue;
-        T* dst = (T*)a.out + (size_t)m * a.hidden + i;
-        float o[VEC];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) o[e] = a.pre.gain ? fmaf(squash<T>(a.pre.alpha * v[r][e]), g[e], s[e]) : v[r][e];
-        if constexpr (VEC == 4) store_four<T>(dst, make_float4(o[0], o[1], o[2], o[3]));
-        else dst[0] = from_float<T>(o[0]);
     }
 }
 

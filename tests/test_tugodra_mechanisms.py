@@ -561,7 +561,7 @@ def test_the_squash_over_its_whole_range():
     for dtype in (torch.float32, torch.bfloat16):
         stream = torch.zeros_like(z).cuda()
         ops.add_tanh_norm(stream, z.cuda(), (1.0, one, nil), 1.0, (1.0, one, nil), dtype)
-        assert float(((stream.cpu().double() - want).abs() / want.abs()).max()) < 1e-6
+        assert float(((stream.cpu().double() - want).abs() / want.abs()).max()) < (1e-6 if dtype == torch.float32 else 4e-6)
 
 
 @pytest.mark.parametrize("device", DEVICES)
