@@ -28,7 +28,7 @@ using namespace mma16;
 
 constexpr int THREADS = 128;
 constexpr int TOK = 64;                    // tokens of a tile
-constexpr int WV = 64, WD = 128;           // value columns and keys of a block of the write kernel
+constexpr int WV = 64, WD = 128, WT = 128; // value columns, keys and tokens of a turn of a block of the write kernel
 constexpr int RV = 128, RD = 64;           // value columns of a block of the read kernel, keys of a staged piece of the state
 constexpr int PAD = 8;                     // an odd number of 16-byte pieces a row: ldmatrix without bank conflicts
 
@@ -123,10 +123,16 @@ __device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, int stride, const
     }
 }
 
-// grid (chunks, heads, ceil(dv / WV) * ceil(d / WD)), block 128: warp w has the 16 value columns w of the block's 64.
+// grid (chunks, heads, ceil(dv / WV) * ceil(d / WD)), block 128: warp w has the 16 value columns w of the block's 64.  WT tokens at a
+// time: a chunk of the usual length is one turn, whose loads are all in flight together.
+struct WriteTile {
+    __nv_bfloat16 k[WT][WD + PAD], vh[WT][WV + PAD], vl[WT][WV + PAD];
+    float w[WT];
+};
+
 __global__ void __launch_bounds__(THREADS) write_kernel(const Args a) {
-    __shared__ __align__(16) __nv_bfloat16 ks[TOK][WD + PAD], vh[TOK][WV + PAD], vl[TOK][WV + PAD];
-    __shared__ float w_s[TOK];
+    extern __shared__ __align__(16) unsigned char smem[];
+    WriteTile& s = *reinterpret_cast<WriteTile*>(smem);
     pdl_wait();
     pdl_launch_dependents();
     const int item = blockIdx.x, head = blockIdx.y, dtiles = (a.d + WD - 1) / WD;
@@ -139,52 +145,67 @@ __global__ void __launch_bounds__(THREADS) write_kernel(const Args a) {
 #pragma unroll
     for (int j = 0; j < WD / 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
     float n_sum = 0.f;
-    for (int t0 = 0; t0 < len; t0 += TOK) {
-        const int n = min(TOK, len - t0);
+    static_assert(WT == THREADS, "a thread a token's weight");
+    constexpr int VPER = WT * (WV / 8) / THREADS;                // 16-byte pieces of values a thread scales
+    for (int t0 = 0; t0 < len; t0 += WT) {
+        const int n = min(WT, len - t0);
         __syncthreads();
-        stage_rows(&ks[0][0], WD + PAD, a.proj + (tok0 + t0) * a.ld + a.k_col + (size_t)head * a.d + d0, a.ld, n, TOK, WD, a.d - d0);
+        stage_rows(&s.k[0][0], WD + PAD, a.proj + (tok0 + t0) * a.ld + a.k_col + (size_t)head * a.d + d0, a.ld, n, WT, WD, a.d - d0);
         cp_async_commit();
-        if (tid < TOK) {
+        const __nv_bfloat16* vsrc = a.proj + (tok0 + t0) * a.ld + a.v_col + (size_t)head * a.dv + v0;
+        uint4 raw[VPER];
+#pragma unroll
+        for (int k = 0; k < VPER; ++k) {
+            const int e = k * THREADS + tid, t = e / (WV / 8), col = (e % (WV / 8)) * 8;
+            raw[k] = t < n && v0 + col < a.dv ? *reinterpret_cast<const uint4*>(vsrc + (size_t)t * a.ld + col) : make_uint4(0, 0, 0, 0);
+        }
+        {
             const size_t at = (tok0 + t0 + (tid < n ? tid : 0)) * a.heads + head;
-            w_s[tid] = tid < n ? expf(a.gate_i[at] - a.gate_b[at] - gmax) : 0.f;
+            s.w[tid] = tid < n ? expf(a.gate_i[at] - a.gate_b[at] - gmax) : 0.f;
         }
         __syncthreads();
-        const __nv_bfloat16* vsrc = a.proj + (tok0 + t0) * a.ld + a.v_col + (size_t)head * a.dv + v0;
-        for (int e = tid; e < TOK * (WV / 8); e += THREADS) {
-            const int t = e / (WV / 8), col = (e % (WV / 8)) * 8;
-            uint4 raw = make_uint4(0, 0, 0, 0);
-            if (t < n && v0 + col < a.dv) raw = *reinterpret_cast<const uint4*>(vsrc + (size_t)t * a.ld + col);
-            const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
-            uint4 hi, lo;
-            uint32_t* h4 = reinterpret_cast<uint32_t*>(&hi);
-            uint32_t* l4 = reinterpret_cast<uint32_t*>(&lo);
-            const float w = w_s[t];
 #pragma unroll
-            for (int k = 0; k < 4; ++k) {
-                const float2 f = __bfloat1622float2(p[k]);
-                split2(f.x * w, f.y * w, h4[k], l4[k]);
-            }
-            *reinterpret_cast<uint4*>(&vh[t][col]) = hi;
-            *reinterpret_cast<uint4*>(&vl[t][col]) = lo;
+        for (int k = 0; k < VPER; ++k) {
+            const int e = k * THREADS + tid, t = e / (WV / 8), col = (e % (WV / 8)) * 8;
+            const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw[k]);
+            uint4 hi, lo;
+            const float w = s.w[t];
+            const float2 f0 = __bfloat1622float2(p[0]), f1 = __bfloat1622float2(p[1]), f2 = __bfloat1622float2(p[2]), f3 = __bfloat1622float2(p[3]);
+            split2(f0.x * w, f0.y * w, hi.x, lo.x);
+            split2(f1.x * w, f1.y * w, hi.y, lo.y);
+            split2(f2.x * w, f2.y * w, hi.z, lo.z);
+            split2(f3.x * w, f3.y * w, hi.w, lo.w);
+            *reinterpret_cast<uint4*>(&s.vh[t][col]) = hi;
+            *reinterpret_cast<uint4*>(&s.vl[t][col]) = lo;
         }
         cp_async_wait<0>();
         __syncthreads();
         if (v0 == 0)
-            for (int t = 0; t < n; ++t) n_sum = fmaf(w_s[t], __bfloat162float(ks[t][tid]), n_sum);
-#pragma unroll
-        for (int k16 = 0; k16 < TOK / 16; ++k16) {
+            for (int t = 0; t < n; ++t) n_sum = fmaf(s.w[t], __bfloat162float(s.k[t][tid]), n_sum);
+        const int steps = (n + 15) / 16;
+        for (int k16 = 0; k16 < steps; ++k16) {
             uint32_t ah[4], al[4];
             const int ar = k16 * 16 + (lane & 7) + ((lane >> 4) << 3), ac = warp * 16 + (((lane >> 3) & 1) << 3);
-            ldmatrix_x4_trans(smem_u32(&vh[ar][ac]), ah[0], ah[1], ah[2], ah[3]);
-            ldmatrix_x4_trans(smem_u32(&vl[ar][ac]), al[0], al[1], al[2], al[3]);
+            ldmatrix_x4_trans(smem_u32(&s.vh[ar][ac]), ah[0], ah[1], ah[2], ah[3]);
+            ldmatrix_x4_trans(smem_u32(&s.vl[ar][ac]), al[0], al[1], al[2], al[3]);
+            // the two parts of a sum are a run of products apart, so that no product waits for the one before it
 #pragma unroll
-            for (int jp = 0; jp < WD / 16; ++jp) {
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4_trans(smem_u32(&ks[k16 * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)][jp * 16 + ((lane >> 4) << 3)]), b0, b1, b2, b3);
-                mma_bf16(acc[2 * jp], ah, b0, b1);
-                mma_bf16(acc[2 * jp + 1], ah, b2, b3);
-                mma_bf16(acc[2 * jp], al, b0, b1);
-                mma_bf16(acc[2 * jp + 1], al, b2, b3);
+            for (int half = 0; half < WD / 64; ++half) {
+                uint32_t b[4][4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u)
+                    ldmatrix_x4_trans(smem_u32(&s.k[k16 * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)][half * 64 + u * 16 + ((lane >> 4) << 3)]),
+                                      b[u][0], b[u][1], b[u][2], b[u][3]);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    mma_bf16(acc[half * 8 + 2 * u], ah, b[u][0], b[u][1]);
+                    mma_bf16(acc[half * 8 + 2 * u + 1], ah, b[u][2], b[u][3]);
+                }
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    mma_bf16(acc[half * 8 + 2 * u], al, b[u][0], b[u][1]);
+                    mma_bf16(acc[half * 8 + 2 * u + 1], al, b[u][2], b[u][3]);
+                }
             }
         }
     }
@@ -250,7 +271,7 @@ __global__ void __launch_bounds__(256) combine_kernel(const Args a) {
 }
 
 // grid (tiles of 64 tokens, heads, ceil(dv / RV)), block 128: warp w has the tokens 16 w ... of the tile.  Shared memory: queries
-// [64][d + PAD], then either pieces of the starting state (two of [RV][RD + PAD]) or keys [64][d + PAD] and values [64][RV + PAD].
+// [64][d + PAD], then either pieces of the starting state (two stages of two of [RV][RD + PAD]) or keys [64][d + PAD] and values [64][RV + PAD].
 __global__ void __launch_bounds__(THREADS) read_kernel(const Args a) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float row_b[TOK], row_m[TOK], key_s[TOK];
@@ -259,7 +280,7 @@ __global__ void __launch_bounds__(THREADS) read_kernel(const Args a) {
     const int d = a.d, dv = a.dv, qstride = d + PAD;
     __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
     __nv_bfloat16* rest = q_s + TOK * qstride;
-    __nv_bfloat16 *hi_s = rest, *lo_s = rest + RV * (RD + PAD), *k_s = rest, *v_s = rest + TOK * qstride;
+    __nv_bfloat16 *k_s = rest, *v_s = rest + TOK * qstride;
     const int tile = gridDim.x - 1 - blockIdx.x;                     // the last tiles of a chunk, which see the most keys, go first
     const int item = a.tile_item[tile], start = a.tile_start[tile], head = blockIdx.y, v0 = blockIdx.z * RV;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c = lane & 3;
@@ -281,30 +302,44 @@ __global__ void __launch_bounds__(THREADS) read_kernel(const Args a) {
 
     // ---- what the starting state answers
     const __nv_bfloat16* qrow = q_s + (warp * 16 + (lane & 15)) * qstride + ((lane >> 4) << 3);
-    for (int d0 = 0; d0 < d; d0 += RD) {
-        __syncthreads();
-        const size_t from = (at * dv + v0) * d + d0;
-        stage_rows(hi_s, RD + PAD, a.start_hi + from, d, dv - v0, RV, RD, d - d0);
-        stage_rows(lo_s, RD + PAD, a.start_lo + from, d, dv - v0, RV, RD, d - d0);
+    auto ask_piece = [&](int k) {                                    // the keys [k RD, (k + 1) RD) of the starting state, stage k % 2
+        const size_t from = (at * dv + v0) * d + k * RD;
+        __nv_bfloat16* to = rest + (k & 1) * 2 * RV * (RD + PAD);
+        stage_rows(to, RD + PAD, a.start_hi + from, d, dv - v0, RV, RD, d - k * RD);
+        stage_rows(to + RV * (RD + PAD), RD + PAD, a.start_lo + from, d, dv - v0, RV, RD, d - k * RD);
         cp_async_commit();
-        cp_async_wait<0>();
-        __syncthreads();
-        const int steps = min(RD, d - d0) / 16;
+    };
+    const int pieces = (d + RD - 1) / RD;
+    ask_piece(0);
+    for (int k = 0; k < pieces; ++k) {
+        if (k + 1 < pieces) {
+            ask_piece(k + 1);
+            cp_async_wait<1>();
+        } else {
+            cp_async_wait<0>();
+        }
+        __syncthreads();                                             // piece k (and the queries) have landed
+        const __nv_bfloat16 *hi_s = rest + (k & 1) * 2 * RV * (RD + PAD), *lo_s = hi_s + RV * (RD + PAD);
+        const int d0 = k * RD, steps = min(RD, d - d0) / 16;
         for (int kk = 0; kk < steps; ++kk) {
             uint32_t q[4];
             ldmatrix_x4(smem_u32(qrow + d0 + kk * 16), q[0], q[1], q[2], q[3]);
             const int br = (lane & 7) + ((lane >> 4) << 3), bc = kk * 16 + (((lane >> 3) & 1) << 3);
+            // the two parts of a sum are a run of products apart, so that no product waits for the one before it
 #pragma unroll
-            for (int jp = 0; jp < RV / 16; ++jp) {
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4(smem_u32(hi_s + (jp * 16 + br) * (RD + PAD) + bc), b0, b1, b2, b3);
-                mma_bf16(o[2 * jp], q, b0, b1);
-                mma_bf16(o[2 * jp + 1], q, b2, b3);
-                ldmatrix_x4(smem_u32(lo_s + (jp * 16 + br) * (RD + PAD) + bc), b0, b1, b2, b3);
-                mma_bf16(o[2 * jp], q, b0, b1);
-                mma_bf16(o[2 * jp + 1], q, b2, b3);
+            for (int part = 0; part < 4; ++part) {
+                const __nv_bfloat16* from = (part & 1 ? lo_s : hi_s) + ((part >> 1) * 64 + br) * (RD + PAD) + bc;
+                uint32_t b[4][4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u) ldmatrix_x4(smem_u32(from + u * 16 * (RD + PAD)), b[u][0], b[u][1], b[u][2], b[u][3]);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    mma_bf16(o[(part >> 1) * 8 + 2 * u], q, b[u][0], b[u][1]);
+                    mma_bf16(o[(part >> 1) * 8 + 2 * u + 1], q, b[u][2], b[u][3]);
+                }
             }
         }
+        __syncthreads();                                             // everyone is done with its stage
     }
     const int r_lo = warp * 16 + g, r_hi = r_lo + 8;
     const float b_lo = row_b[r_lo], b_hi = row_b[r_hi], m_lo = row_m[r_lo], m_hi = row_m[r_hi];
@@ -379,13 +414,21 @@ __global__ void __launch_bounds__(THREADS) read_kernel(const Args a) {
             split2(s[2 * k16 + 1][2], s[2 * k16 + 1][3], ph[3], pl[3]);
             const int vr = k16 * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
 #pragma unroll
-            for (int jp = 0; jp < RV / 16; ++jp) {
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4_trans(smem_u32(v_s + vr * (RV + PAD) + jp * 16 + ((lane >> 4) << 3)), b0, b1, b2, b3);
-                mma_bf16(o[2 * jp], ph, b0, b1);
-                mma_bf16(o[2 * jp + 1], ph, b2, b3);
-                mma_bf16(o[2 * jp], pl, b0, b1);
-                mma_bf16(o[2 * jp + 1], pl, b2, b3);
+            for (int half = 0; half < RV / 64; ++half) {
+                uint32_t b[4][4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u)
+                    ldmatrix_x4_trans(smem_u32(v_s + vr * (RV + PAD) + half * 64 + u * 16 + ((lane >> 4) << 3)), b[u][0], b[u][1], b[u][2], b[u][3]);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    mma_bf16(o[half * 8 + 2 * u], ph, b[u][0], b[u][1]);
+                    mma_bf16(o[half * 8 + 2 * u + 1], ph, b[u][2], b[u][3]);
+                }
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    mma_bf16(o[half * 8 + 2 * u], pl, b[u][0], b[u][1]);
+                    mma_bf16(o[half * 8 + 2 * u + 1], pl, b[u][2], b[u][3]);
+                }
             }
         }
     }
@@ -414,7 +457,7 @@ __global__ void __launch_bounds__(THREADS) read_kernel(const Args a) {
 }
 
 static size_t read_smem(int d) {
-    const size_t q = (size_t)TOK * (d + PAD), pieces = 2 * (size_t)RV * (RD + PAD), tiles = (size_t)TOK * (d + PAD) + (size_t)TOK * (RV + PAD);
+    const size_t q = (size_t)TOK * (d + PAD), pieces = 4 * (size_t)RV * (RD + PAD), tiles = (size_t)TOK * (d + PAD) + (size_t)TOK * (RV + PAD);
     return sizeof(__nv_bfloat16) * (q + (pieces > tiles ? pieces : tiles));
 }
 
@@ -468,7 +511,13 @@ LILY_API int lily_mlstm_chunks(const void* proj, int ld, int q_col, int k_col, i
     launch_pdl(mlc::gates_kernel, dim3(items, (heads + 3) / 4), dim3(mlc::THREADS), 0, stream, a);
     LILY_CHECK_LAUNCH("mlstm_chunk_gates");
     const int wz = (dv + mlc::WV - 1) / mlc::WV * ((d + mlc::WD - 1) / mlc::WD);
-    launch_pdl(mlc::write_kernel, dim3(items, heads, wz), dim3(mlc::THREADS), 0, stream, a);
+    static bool room = false;
+    if (!room) {
+        cudaError_t e = cudaFuncSetAttribute(mlc::write_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(mlc::WriteTile));
+        if (e != cudaSuccess) { set_error("mlstm_chunks: cannot get %zu bytes of shared memory: %s", sizeof(mlc::WriteTile), cudaGetErrorString(e)); return 2; }
+        room = true;
+    }
+    launch_pdl(mlc::write_kernel, dim3(items, heads, wz), dim3(mlc::THREADS), sizeof(mlc::WriteTile), stream, a);
     LILY_CHECK_LAUNCH("mlstm_chunk_write");
     launch_pdl(mlc::combine_kernel, dim3(((dv + 1) * d + 1023) / 1024, heads, longs), dim3(256), 0, stream, a);
     LILY_CHECK_LAUNCH("mlstm_chunk_combine");
