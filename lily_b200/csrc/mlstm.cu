@@ -173,53 +173,73 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_scan_kernel(const MlstmArgs 
 }
 
 // out[t, c] = o / rms(o of the head) * gain[c] * sigmoid(gate[t, c]) with o = y / (max(|nq|, exp(-m)) + floor).
-// grid (tokens, ceil(heads / 4)), block 128: a warp a head of a token.  VEC 4: dv a multiple of four, everything aligned.
-template <typename T, int VEC>
+// VEC 4: dv a multiple of four, everything aligned.  WIDE 0: grid (tokens, ceil(heads / 4)), block 128, a warp a head of a token.
+// WIDE 1 (a few tokens, VEC 4): grid (tokens, heads), block 128, four columns a thread and turn, so that a head's numbers
+// are all asked for together.
+template <typename T, int VEC, int WIDE>
 __global__ void mlstm_out_kernel(const float* __restrict__ y, const float* __restrict__ nq, const float* __restrict__ m, const Operand gate,
                                  int gate_ld, int gate_col, const float* __restrict__ gain, float floor_, float eps, T* __restrict__ out,
                                  float* __restrict__ state, size_t state_stride, size_t m_off, const int* __restrict__ cu_seqlens,
                                  const int* __restrict__ token_req, const int* __restrict__ slots, int heads, int dv) {
+    __shared__ float sums[4];
     pdl_enter_small();
-    const int t = blockIdx.x, head = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int t = blockIdx.x, head = WIDE ? (int)blockIdx.y : blockIdx.y * 4 + (threadIdx.x >> 5), lane = WIDE ? threadIdx.x : threadIdx.x & 31;
     if (head >= heads) return;
+    constexpr int STEP = (WIDE ? 128 : 32) * VEC;
     const size_t at = (size_t)t * heads + head;
+    const float* yr = y + at * dv;
+    const size_t g0 = (size_t)t * gate_ld + gate_col + (size_t)head * dv;
+    const float* gn = gain + (size_t)head * dv;
+    T* dst = out + at * dv;
+    const float4 nil = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 v0 = nil, z0 = nil, w0 = nil;
+    if (WIDE && lane * 4 < dv) {
+        v0 = *reinterpret_cast<const float4*>(yr + lane * 4);
+        z0 = gate.four(g0 + lane * 4);
+        w0 = *reinterpret_cast<const float4*>(gn + lane * 4);
+    }
     const float mt = m[at];
     const int r = token_req[t];
-    if (lane == 0 && t == cu_seqlens[r + 1] - 1) state[(size_t)slots[r] * state_stride + m_off + head] = mt;
     const float inv_den = 1.f / (fmaxf(fabsf(nq[at]), expf(-mt)) + floor_);
-    const float* yr = y + at * dv;
+    auto square = [&](const float4& u) {
+        const float x0 = u.x * inv_den, x1 = u.y * inv_den, x2 = u.z * inv_den, x3 = u.w * inv_den;
+        return x0 * x0 + x1 * x1 + x2 * x2 + x3 * x3;
+    };
     float ssq = 0.f;
     if (VEC == 4) {
-        for (int c = lane * 4; c < dv; c += 128) {
-            const float4 v = *reinterpret_cast<const float4*>(yr + c);
-            const float x = v.x * inv_den, z = v.y * inv_den, u = v.z * inv_den, w = v.w * inv_den;
-            ssq += x * x + z * z + u * u + w * w;
-        }
+        if (WIDE) ssq = square(v0);
+        for (int c = lane * 4 + (WIDE ? STEP : 0); c < dv; c += STEP) ssq += square(*reinterpret_cast<const float4*>(yr + c));
     } else {
         for (int c = lane; c < dv; c += 32) {
             const float x = yr[c] * inv_den;
             ssq = fmaf(x, x, ssq);
         }
     }
-    const float f = inv_den * rsqrtf(warp_sum(ssq) / (float)dv + eps);
-    const size_t g0 = (size_t)t * gate_ld + gate_col + (size_t)head * dv;
-    const float* gn = gain + (size_t)head * dv;
-    T* dst = out + at * dv;
-    if (VEC == 4) {
-        for (int c = lane * 4; c < dv; c += 128) {
-            const float4 v = *reinterpret_cast<const float4*>(yr + c), w = *reinterpret_cast<const float4*>(gn + c), g = gate.four(g0 + c);
-            const float o0 = v.x * f * w.x / (1.f + expf(-g.x)), o1 = v.y * f * w.y / (1.f + expf(-g.y));
-            const float o2 = v.z * f * w.z / (1.f + expf(-g.z)), o3 = v.w * f * w.w / (1.f + expf(-g.w));
-            if constexpr (sizeof(T) == 4) {
-                *reinterpret_cast<float4*>(dst + c) = make_float4(o0, o1, o2, o3);
-            } else {
-                const __nv_bfloat162 lo = __floats2bfloat162_rn(o0, o1), hi = __floats2bfloat162_rn(o2, o3);
-                *reinterpret_cast<uint2*>(dst + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
-            }
+    ssq = warp_sum(ssq);
+    if (WIDE) {
+        if ((threadIdx.x & 31) == 0) sums[threadIdx.x >> 5] = ssq;
+        __syncthreads();
+        ssq = (sums[0] + sums[1]) + (sums[2] + sums[3]);
+    }
+    const float f = inv_den * rsqrtf(ssq / (float)dv + eps);
+    auto finish = [&](int c, const float4& u, const float4& z, const float4& x) {
+        const float o0 = u.x * f * x.x / (1.f + expf(-z.x)), o1 = u.y * f * x.y / (1.f + expf(-z.y));
+        const float o2 = u.z * f * x.z / (1.f + expf(-z.z)), o3 = u.w * f * x.w / (1.f + expf(-z.w));
+        if constexpr (sizeof(T) == 4) {
+            *reinterpret_cast<float4*>(dst + c) = make_float4(o0, o1, o2, o3);
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(o0, o1), hi = __floats2bfloat162_rn(o2, o3);
+            *reinterpret_cast<uint2*>(dst + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
         }
+    };
+    if (VEC == 4) {
+        if (WIDE && lane * 4 < dv) finish(lane * 4, v0, z0, w0);
+        for (int c = lane * 4 + (WIDE ? STEP : 0); c < dv; c += STEP)
+            finish(c, *reinterpret_cast<const float4*>(yr + c), gate.four(g0 + c), *reinterpret_cast<const float4*>(gn + c));
     } else {
         for (int c = lane; c < dv; c += 32) dst[c] = from_float<T>(yr[c] * f * gn[c] / (1.f + expf(-gate(g0 + c))));
     }
+    if (lane == 0 && t == cu_seqlens[r + 1] - 1) state[(size_t)slots[r] * state_stride + m_off + head] = mt;
 }
 
 }  // namespace lily
@@ -276,12 +296,13 @@ LILY_API int lily_mlstm_out(const float* y, const float* nq, const float* m, con
     const Operand g{gate, gate_dtype == kBF16, gate_splits, gate_stride};
     const bool vec = dv % 4 == 0 && gate_ld % 4 == 0 && gate_col % 4 == 0 && g.vector_ok() && ((uintptr_t)y & 15) == 0 &&
                      ((uintptr_t)gain & 15) == 0 && ((uintptr_t)out & 15) == 0;
-    dim3 grid(tokens, (heads + 3) / 4), block(128);
-#define GO(T, V)                                                                                                                       \
-    launch_pdl(mlstm_out_kernel<T, V>, grid, block, 0, stream, y, nq, m, g, gate_ld, gate_col, gain, floor_, eps, (T*)out, state, state_stride, \
+    const bool wide = vec && tokens <= 64 && heads <= 65535;
+    dim3 grid(tokens, wide ? heads : (heads + 3) / 4), block(128);
+#define GO(T, V, W)                                                                                                                    \
+    launch_pdl(mlstm_out_kernel<T, V, W>, grid, block, 0, stream, y, nq, m, g, gate_ld, gate_col, gain, floor_, eps, (T*)out, state, state_stride, \
                m_off, cu_seqlens, token_req, slots, heads, dv)
-    if (out_dtype == kBF16) { if (vec) GO(__nv_bfloat16, 4); else GO(__nv_bfloat16, 1); }
-    else { if (vec) GO(float, 4); else GO(float, 1); }
+    if (out_dtype == kBF16) { if (wide) GO(__nv_bfloat16, 4, 1); else if (vec) GO(__nv_bfloat16, 4, 0); else GO(__nv_bfloat16, 1, 0); }
+    else { if (wide) GO(float, 4, 1); else if (vec) GO(float, 4, 0); else GO(float, 1, 0); }
 #undef GO
     LILY_CHECK_LAUNCH("mlstm_out");
     return 0;

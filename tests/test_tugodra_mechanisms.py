@@ -99,7 +99,7 @@ def attention_part(c, width, eps, w, device, dtype, page, own=True):
 
 
 @pytest.mark.parametrize("device", DEVICES)
-@pytest.mark.parametrize("heads,kv_heads,d,dv,dims", [(3, 1, 12, 12, 12), (4, 2, 64, 64, 64), (6, 2, 64, 64, 32), (2, 2, 128, 128, 128),
+@pytest.mark.parametrize("heads,kv_heads,d,dv,dims", [(3, 1, 12, 12, 12), (4, 2, 64, 64, 64), (8, 2, 64, 64, 32), (2, 2, 128, 128, 128),
                                                       (5, 5, 20, 7, 8), (20, 1, 64, 64, 64), (2, 1, 6, 40, 6)])
 @pytest.mark.parametrize("window,other,page", [(40, 17, 16), (16, 90, 64), (1, 64, 16)])
 def test_windowed_attention_with_keys_that_stand_out(device, heads, kv_heads, d, dv, dims, window, other, page):
@@ -298,8 +298,8 @@ def run_mlstm(part, seqs, plan, device, dtype, slots=None):
     return {k: torch.cat(o) for k, o in outs.items()}, state
 
 
-MLSTM_SIZES = [(2, 8, 12, 10.0), (3, 20, 5, 2.0), (1, 64, 64, 15.0), (4, 32, 48, 12.0), (2, 48, 96, 8.0), (1, 256, 128, 15.0), (2, 144, 136, 6.0),
-               (1, 7, 33, 20.0), (1, 512, 24, 15.0)]
+MLSTM_SIZES = [(2, 8, 12, 10.0), (3, 20, 5, 2.0), (1, 64, 64, 15.0), (5, 32, 40, 11.0), (2, 48, 96, 8.0), (1, 256, 128, 15.0), (2, 144, 136, 6.0),
+               (1, 7, 33, 20.0), (1, 512, 24, 15.0), (1, 16, 640, 15.0)]
 
 
 @pytest.mark.parametrize("device", DEVICES)
@@ -364,7 +364,7 @@ def test_a_value_written_long_ago(device):
 def test_the_scale_starts_at_zero_and_is_carried(device):
     """With input gates far below zero the running maximum stays at what the forget gates leave of its start, zero, and the
     denominator is exp(-m), not |n . q|; the slot carries it from step to step."""
-    c = {"heads": 2, "dim": 16, "vdim": 8, "gate_cap": 12.0}
+    c = {"heads": 2, "dim": 16, "vdim": 8, "gate_cap": 9.0}
     width = 20
     g = torch.Generator().manual_seed(3)
     w = mlstm_weights(g, width, c)
@@ -372,7 +372,7 @@ def test_the_scale_starts_at_zero_and_is_carried(device):
     h = torch.randn(90, width, generator=g)
     part = mlstm_part(c, width, 1e-6, w, device, torch.float32)
     want = pt.mlstm_mixer(h, w, "p", c, 1e-6)
-    i, f = pt.mlstm_gates(h, w, "p", 12.0)
+    i, f = pt.mlstm_gates(h, w, "p", 9.0)
     m, low = torch.zeros(2), []
     for t in range(90):
         m = torch.maximum(f[t] + m, i[t])
@@ -433,7 +433,7 @@ class _Batch:
 
 
 @pytest.mark.parametrize("device", DEVICES)
-@pytest.mark.parametrize("experts,top,groups,keep,ff,width,shared", [(6, 2, 3, 2, 24, 40, 56), (12, 3, 4, 3, 64, 72, None), (4, 1, 2, 1, 10, 33, 7),
+@pytest.mark.parametrize("experts,top,groups,keep,ff,width,shared", [(6, 2, 3, 2, 24, 40, 56), (15, 4, 5, 2, 56, 72, None), (4, 1, 2, 1, 10, 33, 7),
                                                                      (5, 2, 5, 3, 16, 48, 24), (8, 8, 1, 1, 7, 20, 9), (256, 8, 8, 4, 8, 64, 64),
                                                                      (96, 6, 48, 5, 16, 256, 256), (9, 4, None, 1, 32, 64, 40)])
 def test_experts_chosen_within_groups(device, experts, top, groups, keep, ff, width, shared):
